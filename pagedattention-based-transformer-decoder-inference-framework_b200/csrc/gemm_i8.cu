@@ -10,7 +10,7 @@
 // (a split of) K and computes ALL rows of M against it (two 128-row accumulators in TMEM).
 //
 // Pipeline (one CTA per SM, 192 threads):
-//   warp 0   : TMA producer -- cp.async.bulk.tensor (UTMALDG) of A tiles [128 x 128 B] (K-major,
+//   warp 0   : TMA producer -- cp.async.bulk.tensor of A tiles [128 x 128 B] (K-major,
 //              128B swizzle) and the B tile [128 k-rows x 128 B] (N contiguous = "MN-major",
 //              128B swizzle) into a 4-stage shared-memory ring, mbarrier complete_tx.
 //   warp 1   : allocates TMEM, one elected lane issues tcgen05.mma.cta_group::1.kind::i8
@@ -269,7 +269,7 @@ gemm_i8_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
 #endif
 
     if (warp == 0) {
-        if (elect_one()) {  // elect.sync, not lane == 0: operands stay in uniform registers (pa_common.cuh)
+        if (elect_one()) {  // elect.sync, not lane == 0: the MMAs go out back to back
 #ifdef PA_GEMM_PROBE
             long long pw = 0, t_start = clock64();
 #endif

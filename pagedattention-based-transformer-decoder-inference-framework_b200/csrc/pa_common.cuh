@@ -117,10 +117,9 @@ __device__ __forceinline__ void mbar_wait(uint32_t bar, uint32_t parity) {
     while (!mbar_try_wait(bar, parity)) {
     }
 }
-// One lane of a converged warp.  ptxas recognises elect.sync: code under `if (elect_one())` keeps its
-// warp-uniform operands in uniform registers, so consecutive tcgen05.mma / TMA instructions are issued back
-// to back.  Under `if (lane == 0)` every such instruction is wrapped in an R2UR + ELECT + BRA.U.ANY
-// "uniformisation" loop (~100 cycles per instruction, measured with clock64 probes in prefill_tc.cu).
+// One lane of a converged warp, by elect.sync.  Consecutive tcgen05.mma / TMA instructions under
+// `if (elect_one())` are issued back to back; under `if (lane == 0)` each of them took ~100 cycles
+// (measured with clock64 probes in prefill_tc.cu).
 __device__ __forceinline__ bool elect_one() {
     uint32_t pred;
     asm volatile(

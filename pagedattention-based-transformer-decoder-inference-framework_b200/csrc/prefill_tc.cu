@@ -389,8 +389,7 @@ __global__ void __launch_bounds__(threads_for(KV, NQ, MW), (NQ == 1 && KV == 0) 
     } else if (warp == W_PROD) {
         // ------------------------------------------------------------ TMA producer
         // ONE elected thread issues the 16 boxes of a tile (unit uu x {K lo, K hi, V lo, V hi}).  Everything
-        // under elect_one() stays in uniform registers, so the 16 UTMALDG go out back to back; page ids are
-        // fetched one tile ahead.
+        // is under elect_one(), so the 16 copies go out back to back; page ids are fetched one tile ahead.
         if (elect_one()) {
             int pgn[4];
             auto load_pages = [&](int tile) {
