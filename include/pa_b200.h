@@ -810,6 +810,59 @@ int pa_gated_rms_norm(const float* d_y, int64_t rows, int inner, int groups, con
                       int gate_off, int gate_mode, const float* d_weight, float eps, void* d_out, int elem,
                       pa_stream_t stream);
 
+/* ---- sigmoid weights, keys as values, rotated retention, residual streams -------------------------------------------
+ * pa_masked_attention_gated: pa_masked_attention_sink with: d_key_scale [total_pages * tile_size] (NULL: none), a factor
+ *   per pool row on the dot product; sigmoid_weights 1: the weight of a visible key is sigmoid(score) and nothing divides
+ *   the sum (no sink then); d_head_bias [heads] (NULL: none) added to the score last; d_gate (NULL: none): rows of the
+ *   activation type, output column c of head h is multiplied by sigmoid(gate[row * gate_stride + gate_off + h * vdim + c])
+ *   in float before it is rounded.  d_v_pool == d_k_pool (dim == vdim): the values are the cached key rows, read once.
+ * pa_qk_norm_kv_append: query head h (columns q_off + h * dim) is divided by its root mean square and multiplied by
+ *   d_q_gain [dim], in place; the key of kv head g (k_off + g * dim) goes to the row's place in the pool: normed likewise
+ *   (d_k_gain) where d_key_scale is NULL, else as it is, with its inverse root mean square in d_key_scale (the key norm's
+ *   gain is then part of d_q_gain).  d_v_pool (NULL: none): the value row (v_off + g * vdim) as it is.
+ * pa_decay_scan_rotated: pa_decay_scan where q and k are rotated over their first rot_dims dimensions (pairs
+ *   (i, i + rot_dims / 2), d_rope [rows][rot_dims / 2][cos, sin]) and k is multiplied by k_scale (constant decays), in float.
+ *   pa_gated_rms_norm also takes d_weight NULL (ones) and gate_mode 3 (the result times silu(gate)).
+ * pa_rope_rows_paired: pa_rope_rows with the pairs chosen: 0 neighbours (2i, 2i + 1), 1 halves (i, i + dims / 2).
+ * pa_latent_norm_append: pa_latent_kv_append with the pairs chosen, and, where d_q_out is given, in the same launch
+ *   q_out[r] = RMS norm of the row's q_rank columns at q_off times d_q_gain.
+ * pa_streams_add_norm: a residual of `streams` float rows per token, x_s (d_src [rows][src_streams][width]; src_streams 1:
+ *   every stream is the one row): x'_t = sum_s d_mix[s][t] x_s + d_out_w[t] y (d_y and d_mix NULL: x' = x), kept in d_dst
+ *   [rows][streams][width] (may be d_src; NULL: not kept); u = sum_t d_in_w[t] x'_t (NULL: ones) to d_u (float, optional)
+ *   and u / sqrt(mean(u^2) + eps) * d_gain to d_next (activation type, optional).  d_row_ids (NULL: all rows): output row
+ *   r is batch row d_row_ids[r] (d_dst must be NULL).  At most 16 streams. */
+int pa_masked_attention_gated(const void* d_q, int64_t q_stride, int q_off, const void* d_k_pool, const void* d_v_pool,
+                              const int32_t* d_table, int num_slots, int num_kv_heads, int num_tiles, int total_pages,
+                              int tile_size, const int32_t* d_q_tiles, int num_q_tiles, int heads, int dim, int vdim,
+                              float scale, float softcap, int mask_kind, int mask_size, int mask_keep, int bias_kind,
+                              const float* d_bias, int bias_len, const float* d_head_scale, const float* d_sink,
+                              const float* d_out_rot, const float* d_key_scale, int sigmoid_weights,
+                              const float* d_head_bias, const void* d_gate, int64_t gate_stride, int gate_off, void* d_out,
+                              int elem, int tile_kind, pa_stream_t stream);
+int pa_qk_norm_kv_append(void* d_src, int64_t src_stride, int q_off, int k_off, int v_off, int heads, int kv_heads, int dim,
+                         int vdim, const float* d_q_gain, const float* d_k_gain, float eps, void* d_k_pool, void* d_v_pool,
+                         float* d_key_scale, const int32_t* d_table, int num_slots, int num_tiles, int total_pages,
+                         int tile_size, const int32_t* d_row_slot, const int32_t* d_row_pos, int rows, int elem,
+                         pa_stream_t stream);
+int pa_decay_scan_rotated(const void* d_q, int64_t q_stride, int q_off, const void* d_k, int64_t k_stride, int k_off,
+                          const void* d_v, int64_t v_stride, int v_off, int heads, int groups, int dim, int vdim, int act,
+                          const float* d_decay, const void* d_dt, int64_t dt_stride, int dt_off, const float* d_dt_bias,
+                          const float* d_a_log, const float* d_skip, const float* d_rope, int rot_dims, float k_scale,
+                          float* d_state, float* d_out, int64_t out_stride, const int32_t* d_items, int num_items,
+                          const int32_t* d_seq_chunk0, const int32_t* d_seq_nchunks, const int32_t* d_seq_slot, int num_seqs,
+                          int chunked, void* d_workspace, size_t workspace_bytes, int elem, pa_stream_t stream);
+int pa_rope_rows_paired(void* d_x, int64_t stride, int off, int head_stride, int heads, int dims, const float* d_table,
+                        int pairing, int rows, int elem, pa_stream_t stream);
+int pa_latent_norm_append(void* d_pool, const int32_t* d_table, int num_slots, int num_tiles, int total_pages,
+                          int tile_size, int kv_rank, int rot_dim, int rot_dims, int pairing, const void* d_src,
+                          int64_t src_stride, int c_off, const float* d_gain, float eps, const float* d_rope_table,
+                          int q_off, int q_rank, const float* d_q_gain, void* d_q_out, int64_t q_out_stride,
+                          const int32_t* d_row_slot, const int32_t* d_row_pos, int rows, int elem, pa_stream_t stream);
+int pa_streams_add_norm(const float* d_src, int src_streams, float* d_dst, int64_t rows, int streams, int width,
+                        const void* d_y, const float* d_mix, const float* d_out_w, const float* d_in_w, float eps,
+                        const float* d_gain, float* d_u, void* d_next, const int32_t* d_row_ids, int elem,
+                        pa_stream_t stream);
+
 #ifdef __cplusplus
 }
 #endif

@@ -14,9 +14,10 @@
 // float; pool rows are stored in the activation type (float or bfloat16).
 //
 //   rope_table_kernel        cos / sin of p * base^(-2i / dims) per batch row (angles in double, table in float)
-//   rope_rows_kernel         in-place rotation of interleaved pairs (2i, 2i + 1) of every head's rotated part
+//   rope_rows_kernel         in-place rotation of the pairs of every head's rotated part: (2i, 2i + 1), or halves
+//                            (i, i + dims / 2)
 //   latent_kv_append_kernel  RMS norm (per-channel gain) of the latent columns + rotation of the shared key part, written
-//                            to the row's place in the pool
+//                            to the row's place in the pool; optionally the norm of the query latent in the same launch
 //   head_linear_kernel       out[r, h, :] = x[r, h, :] . W[h]  (W [heads][K][N]), any strides
 //   latent_attention_kernel  float tile kernel, any shape, keys optionally split with a merge kernel
 //   latent_attention_mma_kernel  bfloat16 tensor-core kernel (mma.sync), see there
@@ -39,10 +40,14 @@ __global__ void rope_table_kernel(const int32_t* __restrict__ row_pos, int rows,
     table[2 * i + 1] = (float)s;
 }
 
-// x[r, off + h * head_stride + 2i .. + 1], i < dims / 2, rotated by the row's table entry
+// the two members of pair k of `half` pairs: neighbours (pairing 0) or entry k of either half (pairing 1)
+__device__ __forceinline__ int pair_first(int k, int pairing) { return pairing ? k : 2 * k; }
+__device__ __forceinline__ int pair_second(int k, int half, int pairing) { return pairing ? k + half : 2 * k + 1; }
+
+// the pairs k < dims / 2 from column off + h * head_stride of every row, rotated by the row's table entry
 template <typename T>
 __global__ void rope_rows_kernel(T* __restrict__ x, int64_t stride, int off, int head_stride, int heads, int dims,
-                                 const float* __restrict__ table, int rows) {
+                                 const float* __restrict__ table, int rows, int pairing) {
     const int half = dims / 2;
     const int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= (int64_t)rows * heads * half) return;
@@ -50,23 +55,46 @@ __global__ void rope_rows_kernel(T* __restrict__ x, int64_t stride, int off, int
     const int h = (int)((i / half) % heads);
     const int64_t r = i / ((int64_t)half * heads);
     const float c = table[(r * half + k) * 2], s = table[(r * half + k) * 2 + 1];
-    T* p = x + r * stride + off + (int64_t)h * head_stride + 2 * k;
-    const float u = to_f32<T>(p[0]), v = to_f32<T>(p[1]);
-    p[0] = from_f32<T>(u * c - v * s);
-    p[1] = from_f32<T>(v * c + u * s);
+    T* p = x + r * stride + off + (int64_t)h * head_stride;
+    T* p0 = p + pair_first(k, pairing);
+    T* p1 = p + pair_second(k, half, pairing);
+    const float u = to_f32<T>(*p0), v = to_f32<T>(*p1);
+    *p0 = from_f32<T>(u * c - v * s);
+    *p1 = from_f32<T>(v * c + u * s);
 }
 
-// One warp per row: src row = [.. | c_raw (kv_rank) at c_off | kr_raw (rot_dim) right behind it].
+// RMS norm of a row by one warp
+template <typename T>
+__device__ __forceinline__ void rms_row_warp(const T* __restrict__ s, int width, float eps, const float* __restrict__ gain,
+                                             T* __restrict__ dst, int lane) {
+    float ss = 0.f;
+    for (int d = lane; d < width; d += 32) {
+        const float v = to_f32<T>(s[d]);
+        ss = fmaf(v, v, ss);
+    }
+    ss = warp_sum(ss);
+    const float rn = 1.0f / sqrtf(ss / (float)width + eps);
+    for (int d = lane; d < width; d += 32) dst[d] = from_f32<T>(to_f32<T>(s[d]) * rn * gain[d]);
+}
+
+// One warp per (row, unit): src row = [.. | c_raw (kv_rank) at c_off | kr_raw (rot_dim) right behind it]; unit 0 appends
+// it, unit 1 (units == 2) norms the query latent of the same row: q_rank columns at q_off -> q_out.
 template <typename T>
 __global__ void latent_kv_append_kernel(T* __restrict__ pool, const int32_t* __restrict__ table, int num_slots,
                                         int num_tiles, int total_pages, int tile_size, int kv_rank, int rot_dim,
                                         int rot_dims, const T* __restrict__ src, int64_t src_stride, int c_off,
                                         const float* __restrict__ gain, float eps, const float* __restrict__ rope,
                                         const int32_t* __restrict__ row_slot, const int32_t* __restrict__ row_pos,
-                                        int rows) {
+                                        int rows, int pairing, int units, int q_off, int q_rank,
+                                        const float* __restrict__ q_gain, T* __restrict__ q_out, int64_t q_out_stride) {
     const int lane = threadIdx.x & 31;
-    const int64_t r = ((int64_t)blockIdx.x * blockDim.x + threadIdx.x) >> 5;
-    if (r >= rows) return;
+    const int64_t w = ((int64_t)blockIdx.x * blockDim.x + threadIdx.x) >> 5;
+    if (w >= (int64_t)rows * units) return;
+    const int64_t r = w / units;
+    if (w % units == 1) {
+        rms_row_warp<T>(src + r * src_stride + q_off, q_rank, eps, q_gain, q_out + r * q_out_stride, lane);
+        return;
+    }
     const int slot = row_slot[r], pos = row_pos[r];
     if (pos < 0 || pos / tile_size >= num_tiles || (unsigned)slot >= (unsigned)num_slots) return;
     const int page = table[(int64_t)slot * num_tiles + pos / tile_size];
@@ -74,20 +102,14 @@ __global__ void latent_kv_append_kernel(T* __restrict__ pool, const int32_t* __r
     const int kd = kv_rank + rot_dim;
     T* dst = pool + ((int64_t)page * tile_size + pos % tile_size) * kd;
     const T* s = src + r * src_stride + c_off;
-    float ss = 0.f;
-    for (int d = lane; d < kv_rank; d += 32) {
-        const float v = to_f32<T>(s[d]);
-        ss = fmaf(v, v, ss);
-    }
-    ss = warp_sum(ss);
-    const float rn = 1.0f / sqrtf(ss / (float)kv_rank + eps);
-    for (int d = lane; d < kv_rank; d += 32) dst[d] = from_f32<T>(to_f32<T>(s[d]) * rn * gain[d]);
+    rms_row_warp<T>(s, kv_rank, eps, gain, dst, lane);
     const int half = rot_dims / 2;
     for (int k = lane; k < half; k += 32) {
         const float c = rope[(r * half + k) * 2], sn = rope[(r * half + k) * 2 + 1];
-        const float u = to_f32<T>(s[kv_rank + 2 * k]), v = to_f32<T>(s[kv_rank + 2 * k + 1]);
-        dst[kv_rank + 2 * k] = from_f32<T>(u * c - v * sn);
-        dst[kv_rank + 2 * k + 1] = from_f32<T>(v * c + u * sn);
+        const int i0 = kv_rank + pair_first(k, pairing), i1 = kv_rank + pair_second(k, half, pairing);
+        const float u = to_f32<T>(s[i0]), v = to_f32<T>(s[i1]);
+        dst[i0] = from_f32<T>(u * c - v * sn);
+        dst[i1] = from_f32<T>(v * c + u * sn);
     }
     for (int d = rot_dims + lane; d < rot_dim; d += 32) dst[kv_rank + d] = s[kv_rank + d];   // unrotated remainder
 }
@@ -99,15 +121,7 @@ __global__ void rms_rows_kernel(const T* __restrict__ src, int64_t src_stride, i
     const int lane = threadIdx.x & 31;
     const int64_t r = ((int64_t)blockIdx.x * blockDim.x + threadIdx.x) >> 5;
     if (r >= rows) return;
-    const T* s = src + r * src_stride + off;
-    float ss = 0.f;
-    for (int d = lane; d < width; d += 32) {
-        const float v = to_f32<T>(s[d]);
-        ss = fmaf(v, v, ss);
-    }
-    ss = warp_sum(ss);
-    const float rn = 1.0f / sqrtf(ss / (float)width + eps);
-    for (int d = lane; d < width; d += 32) dst[r * dst_stride + d] = from_f32<T>(to_f32<T>(s[d]) * rn * gain[d]);
+    rms_row_warp<T>(src + r * src_stride + off, width, eps, gain, dst + r * dst_stride, lane);
 }
 
 // ---- per-head products ----------------------------------------------------------------------------------------------
@@ -826,11 +840,16 @@ PA_API int pa_rope_table(const int32_t* d_row_pos, int rows, int dims, float bas
 
 PA_API int pa_rope_rows(void* d_x, int64_t stride, int off, int head_stride, int heads, int dims, const float* d_table,
                         int rows, int elem, pa_stream_t stream) {
-    PA_CHECK_ARG(d_x && d_table && rows >= 0 && heads > 0 && dims >= 0 && dims % 2 == 0);
+    return pa_rope_rows_paired(d_x, stride, off, head_stride, heads, dims, d_table, 0, rows, elem, stream);
+}
+
+PA_API int pa_rope_rows_paired(void* d_x, int64_t stride, int off, int head_stride, int heads, int dims,
+                               const float* d_table, int pairing, int rows, int elem, pa_stream_t stream) {
+    PA_CHECK_ARG(d_x && d_table && rows >= 0 && heads > 0 && dims >= 0 && dims % 2 == 0 && (pairing == 0 || pairing == 1));
     const int64_t n = (int64_t)rows * heads * (dims / 2);
     if (n == 0) return PA_OK;
     PA_DISPATCH_ELEM(elem, rope_rows_kernel<T><<<(unsigned)((n + 255) / 256), 256, 0, as_stream(stream)>>>(
-                               static_cast<T*>(d_x), stride, off, head_stride, heads, dims, d_table, rows));
+                               static_cast<T*>(d_x), stride, off, head_stride, heads, dims, d_table, rows, pairing));
     PA_RETURN_LAUNCH_STATUS();
 }
 
@@ -839,15 +858,29 @@ PA_API int pa_latent_kv_append(void* d_pool, const int32_t* d_table, int num_slo
                                int c_off, const float* d_gain, float eps, const float* d_rope_table,
                                const int32_t* d_row_slot, const int32_t* d_row_pos, int rows, int elem,
                                pa_stream_t stream) {
+    return pa_latent_norm_append(d_pool, d_table, num_slots, num_tiles, total_pages, tile_size, kv_rank, rot_dim, rot_dims, 0,
+                                 d_src, src_stride, c_off, d_gain, eps, d_rope_table, 0, 0, nullptr, nullptr, 0, d_row_slot,
+                                 d_row_pos, rows, elem, stream);
+}
+
+PA_API int pa_latent_norm_append(void* d_pool, const int32_t* d_table, int num_slots, int num_tiles, int total_pages,
+                                 int tile_size, int kv_rank, int rot_dim, int rot_dims, int pairing, const void* d_src,
+                                 int64_t src_stride, int c_off, const float* d_gain, float eps, const float* d_rope_table,
+                                 int q_off, int q_rank, const float* d_q_gain, void* d_q_out, int64_t q_out_stride,
+                                 const int32_t* d_row_slot, const int32_t* d_row_pos, int rows, int elem,
+                                 pa_stream_t stream) {
     PA_CHECK_ARG(d_pool && d_table && d_src && d_gain && d_row_slot && d_row_pos && rows >= 0);
+    PA_CHECK_ARG((pairing == 0 || pairing == 1) && (!d_q_out || (d_q_gain && q_rank > 0)));
     PA_CHECK_ARG(num_slots > 0 && num_tiles > 0 && total_pages > 0 && tile_size > 0 && kv_rank > 0 && rot_dim >= 0);
     PA_CHECK_ARG(rot_dims >= 0 && rot_dims <= rot_dim && rot_dims % 2 == 0 && (rot_dims == 0 || d_rope_table));
     if (rows == 0) return PA_OK;
-    const int64_t threads = (int64_t)rows * 32;
+    const int units = d_q_out ? 2 : 1;
+    const int64_t threads = (int64_t)rows * units * 32;
     PA_DISPATCH_ELEM(elem, latent_kv_append_kernel<T><<<(unsigned)((threads + 255) / 256), 256, 0, as_stream(stream)>>>(
                                static_cast<T*>(d_pool), d_table, num_slots, num_tiles, total_pages, tile_size, kv_rank,
                                rot_dim, rot_dims, static_cast<const T*>(d_src), src_stride, c_off, d_gain, eps,
-                               d_rope_table, d_row_slot, d_row_pos, rows));
+                               d_rope_table, d_row_slot, d_row_pos, rows, pairing, units, q_off, q_rank, d_q_gain,
+                               static_cast<T*>(d_q_out), q_out_stride));
     PA_RETURN_LAUNCH_STATUS();
 }
 

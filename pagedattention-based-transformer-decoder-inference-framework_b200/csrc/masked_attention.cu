@@ -1,4 +1,4 @@
-// masked_attention.cu -- softmax attention with grouped key/value heads over the paged KV pools for a RAGGED batch
+// masked_attention.cu -- softmax or sigmoid attention with grouped key/value heads over the paged KV pools for a RAGGED batch
 // (prompt portions and single decoded tokens in one launch), with the score modifiers and visibility rules a design
 // picks by parameter:
 //
@@ -6,6 +6,10 @@
 //           bias_kind 1: - slope[h] * (i - j)            (one slope per query head)
 //           bias_kind 2: + table[min(i - j, len - 1)][h] (a table over the distance, one column per query head)
 //           head_scale != null: s <- s * head_scale[h] right after the scale (a temperature per query head)
+//           key_scale != null: the dot product is first multiplied by a number per cached key (the inverse root mean
+//           square of a key that is cached before its norm)
+//           head_bias != null: + head_bias[h], last
+//   weight  softmax over the visible keys, or (sigm) sigmoid(s) of every visible key, with no sum to divide by
 //   mask    mask_kind 0: causal (j <= i);  1: sliding window (0 <= i - j < size), which with mask_keep > 0 also keeps the
 //           first mask_keep positions of the sequence visible (at their true positions);  2: chunks (j <= i and
 //           floor(i / size) == floor(j / size), chunks counted from position 0 of the sequence)
@@ -14,6 +18,8 @@
 //   output  out_rot != null: [rows][vdim / 2][cos, sin] of the batch rows; the neighbouring pairs (2m, 2m + 1) of every
 //           head's output are turned BACK by the row's angle (values that were cached turned by their own position), in
 //           float, before the result is rounded
+//           gate != null: multiplied element by element by sigmoid(gate row), in float, before the result is rounded
+//   values  v_pool == k_pool (and vdim == dim): the values ARE the cached key rows; the pool holds one row per key
 //
 
 // No rotation: positions enter through the bias and the mask only.  Scores, the modifiers, softmax weights and the
@@ -77,6 +83,64 @@ __global__ void rope_kv_append_kernel(T* __restrict__ src, int64_t stride, int q
                     vrot ? vrot + r * (vdim >> 1) * 2 : nullptr, lane);
 }
 
+// ---- query / key norm of this step's rows fused with the append --------------------------------------------------------
+// One warp per (row, unit): units [0, heads) are the query heads, divided by their root mean square and multiplied by
+// q_gain, in place; units [heads, heads + kv_heads) are the key/value heads.  key_scale == null: the key goes to its place
+// in the pool normed (k_gain).  key_scale != null: the key goes there as projected and its inverse root mean square to
+// key_scale, so the pool row can serve as the value too (the key norm's gain is then part of q_gain: only the product of
+// the two enters a score).  v_pool != null: a value row of its own, as it is.
+template <typename T>
+__device__ __forceinline__ float qk_inv_rms(const T* __restrict__ x, int dim, float eps, int lane) {
+    float ss = 0.f;
+    for (int d = lane; d < dim; d += 32) {
+        const float v = to_f32<T>(x[d]);
+        ss = fmaf(v, v, ss);
+    }
+    return 1.0f / sqrtf(warp_sum(ss) / (float)dim + eps);
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) qk_norm_kv_append_kernel(T* __restrict__ src, int64_t stride, int q_off, int k_off, int v_off,
+                                         int heads, int kv_heads, int dim, int vdim, const float* __restrict__ q_gain,
+                                         const float* __restrict__ k_gain, float eps, T* __restrict__ k_pool,
+                                         T* __restrict__ v_pool, float* __restrict__ key_scale,
+                                         const int32_t* __restrict__ table, int num_slots, int num_tiles, int total_pages,
+                                         int tile_size, const int32_t* __restrict__ row_slot,
+                                         const int32_t* __restrict__ row_pos, int rows) {
+    const int lane = threadIdx.x & 31;
+    const int units = heads + kv_heads;
+    const int64_t w = ((int64_t)blockIdx.x * blockDim.x + threadIdx.x) >> 5;
+    if (w >= (int64_t)rows * units) return;
+    const int u = (int)(w % units);
+    const int64_t r = w / units;
+    T* row = src + r * stride;
+    if (u < heads) {
+        T* q = row + q_off + (int64_t)u * dim;
+        const float rn = qk_inv_rms<T>(q, dim, eps, lane);
+        for (int d = lane; d < dim; d += 32) q[d] = from_f32<T>(to_f32<T>(q[d]) * rn * q_gain[d]);
+        return;
+    }
+    const int g = u - heads;
+    const int slot = row_slot[r], pos = row_pos[r];
+    if (pos < 0 || pos / tile_size >= num_tiles || (unsigned)slot >= (unsigned)num_slots) return;
+    const int page = table[((int64_t)slot * kv_heads + g) * num_tiles + pos / tile_size];
+    if (page < 0 || page >= total_pages) return;
+    const int64_t prow = (int64_t)page * tile_size + pos % tile_size;
+    const T* k = row + k_off + (int64_t)g * dim;
+    const float rn = qk_inv_rms<T>(k, dim, eps, lane);
+    T* kd = k_pool + prow * dim;
+    if (key_scale) {
+        for (int d = lane; d < dim; d += 32) kd[d] = k[d];
+        if (lane == 0) key_scale[prow] = rn;
+    } else {
+        for (int d = lane; d < dim; d += 32) kd[d] = from_f32<T>(to_f32<T>(k[d]) * rn * k_gain[d]);
+    }
+    if (v_pool) {
+        const T* v = row + v_off + (int64_t)g * vdim;
+        for (int d = lane; d < vdim; d += 32) v_pool[prow * vdim + d] = v[d];
+    }
+}
+
 constexpr int kMaRows = 32;     // (token, head) rows per CTA
 constexpr int kMaWarps = 8;
 constexpr int kMaRpw = kMaRows / kMaWarps;
@@ -102,6 +166,12 @@ struct MaskAttnParams {
     int mask_keep;              // window masks: the first mask_keep positions stay visible
     const float* out_rot;       // [rows][vdim / 2][2] or null
     int head_rows;              // tensor-core kernel: every tile is ONE token and the rows are the heads of a kv head
+    int sigm;                   // 1: weight = sigmoid(score), nothing divides the sum (no sink)
+    const float* key_scale;     // [total_pages * tile_size] or null
+    const float* head_bias;     // [heads] or null
+    const void* gate;           // rows of the activation type; the gate of output column c of head h at gate_off + h * vdim + c
+    int64_t gate_stride;
+    int gate_off;
 };
 
 __device__ __forceinline__ int ma_first_key(const MaskAttnParams& p, int pos) {
@@ -156,7 +226,14 @@ __device__ __forceinline__ float ma_score(const MaskAttnParams& p, float dot, in
     if (p.softcap > 0.f) s = p.softcap * tanhf(s / p.softcap);
     if (p.bias_kind == 1) s -= slope * (float)(i - j);
     else if (p.bias_kind == 2) s += p.bias[(int64_t)min(i - j, p.bias_len - 1) * p.heads + h];
+    if (p.head_bias) s += p.head_bias[h];
     return s;
+}
+
+// the factor of output column `col` (of all heads' columns) of batch row `row`
+template <typename T>
+__device__ __forceinline__ float ma_gate(const MaskAttnParams& p, int64_t row, int col) {
+    return sigmoid_f32(to_f32<T>(static_cast<const T*>(p.gate)[row * p.gate_stride + p.gate_off + col]));
 }
 
 __device__ __forceinline__ void ma_geometry(int heads, int kv_heads, int& hpg, int& hc, int& nchunk) {
@@ -254,11 +331,16 @@ __global__ void __launch_bounds__(kMaWarps * 32) masked_attention_kernel(const M
         }
         const int j = c0 + lane;
         const bool mapped = page_row[lane] >= 0;
+        const float ks = mapped && p.key_scale ? p.key_scale[page_row[lane]] : 1.f;
         float w[kMaRpw];
 #pragma unroll
         for (int r = 0; r < kMaRpw; ++r) {
             const bool vis = mapped && rpos[r] >= 0 && ma_visible(p, rpos[r], j);
-            const float v = vis ? ma_score(p, s[r], rpos[r], j, rhead[r], slope[r]) : -INFINITY;
+            const float v = vis ? ma_score(p, s[r] * ks, rpos[r], j, rhead[r], slope[r]) : -INFINITY;
+            if (p.sigm) {
+                w[r] = vis ? sigmoid_f32(v) : 0.f;
+                continue;
+            }
             const float n = fmaxf(m[r], warp_max(v));
             const float c = n == -INFINITY ? 1.f : expf(m[r] - n);
             w[r] = vis ? expf(v - n) : 0.f;
@@ -288,7 +370,7 @@ __global__ void __launch_bounds__(kMaWarps * 32) masked_attention_kernel(const M
         const int row = warp * kMaRpw + r;
         T* dst = static_cast<T*>(p.out) + (int64_t)(row0 + row / hc) * p.heads * p.vdim + (int64_t)rhead[r] * p.vdim;
         float ll = l[r];
-        const float inv = ma_sink(p, rhead[r], m[r], ll) / ll;
+        const float inv = p.sigm ? 1.f : ma_sink(p, rhead[r], m[r], ll) / ll;
 #pragma unroll
         for (int i = 0; i < NV; ++i) {
             const int col = lane + 32 * i;
@@ -297,6 +379,7 @@ __global__ void __launch_bounds__(kMaWarps * 32) masked_attention_kernel(const M
                 const float o = __shfl_xor_sync(0xffffffffu, v, 1);
                 if (col < p.vdim) v = ma_unturn(p, row0 + row / hc, col, v, o);
             }
+            if (p.gate && col < p.vdim) v *= ma_gate<T>(p, row0 + row / hc, rhead[r] * p.vdim + col);
             if (col < p.vdim) dst[col] = from_f32<T>(v);
         }
     }
@@ -447,10 +530,15 @@ __global__ void __launch_bounds__(kMaDecWarps * 32) masked_attention_decode_kern
             }
         }
         const bool vis = prow >= 0;
+        const float ks = vis && p.key_scale ? p.key_scale[prow] : 1.f;
         float w[R];
 #pragma unroll
         for (int r = 0; r < R; ++r) {
-            const float v = vis && r < hpg ? ma_score(p, s[r], pos, j, g * hpg + r, slope[r]) : -INFINITY;
+            const float v = vis && r < hpg ? ma_score(p, s[r] * ks, pos, j, g * hpg + r, slope[r]) : -INFINITY;
+            if (p.sigm) {
+                w[r] = v == -INFINITY ? 0.f : sigmoid_f32(v);
+                continue;
+            }
             const float n = fmaxf(m[r], warp_max(v));
             const float c = n == -INFINITY ? 1.f : expf(m[r] - n);
             w[r] = v == -INFINITY ? 0.f : expf(v - n);
@@ -498,19 +586,20 @@ __global__ void __launch_bounds__(kMaDecWarps * 32) masked_attention_decode_kern
         float M = -INFINITY;
         for (int w = 0; w < kMaDecWarps; ++w) M = fmaxf(M, Ps[((int64_t)w * R + r) * pstride]);
         if (p.sink) M = fmaxf(M, p.sink[g * hpg + r]);
+        if (p.sigm) M = 0.f;
         float L = p.sink ? expf(p.sink[g * hpg + r] - M) : 0.f, b[NV];
 #pragma unroll
         for (int i = 0; i < NV; ++i) b[i] = 0.f;
         for (int w = 0; w < kMaDecWarps; ++w) {
             const float* pw = Ps + ((int64_t)w * R + r) * pstride;
-            const float f = pw[0] == -INFINITY ? 0.f : expf(pw[0] - M);
+            const float f = p.sigm ? 1.f : pw[0] == -INFINITY ? 0.f : expf(pw[0] - M);
             L = fmaf(f, pw[1], L);
 #pragma unroll
             for (int i = 0; i < NV; ++i)
                 if (ma_col<NV, PACKED>(lane, i) < p.vdim) b[i] = fmaf(f, pw[2 + ma_col<NV, PACKED>(lane, i)], b[i]);
         }
         T* dst = static_cast<T*>(p.out) + (int64_t)row0 * p.heads * p.vdim + (int64_t)(g * hpg + r) * p.vdim;
-        const float inv = 1.0f / L;
+        const float inv = p.sigm ? 1.0f : 1.0f / L;
 #pragma unroll
         for (int i = 0; i < NV; ++i) b[i] *= inv;
         if (p.out_rot) {          // the partner column: the neighbouring slot of this lane (packed pairs) or the neighbouring lane
@@ -520,6 +609,11 @@ __global__ void __launch_bounds__(kMaDecWarps * 32) masked_attention_decode_kern
 #pragma unroll
             for (int i = 0; i < NV; ++i)
                 if (ma_col<NV, PACKED>(lane, i) < p.vdim) b[i] = ma_unturn(p, row0, ma_col<NV, PACKED>(lane, i), b[i], o[i]);
+        }
+        if (p.gate) {
+#pragma unroll
+            for (int i = 0; i < NV; ++i)
+                if (ma_col<NV, PACKED>(lane, i) < p.vdim) b[i] *= ma_gate<T>(p, row0, (g * hpg + r) * p.vdim + ma_col<NV, PACKED>(lane, i));
         }
 #pragma unroll
         for (int i = 0; i < NV; ++i)
@@ -572,7 +666,8 @@ static int ma_decode_dispatch(const MaskAttnParams& p, int ntiles, cudaStream_t 
 // the weights enter the second product rounded to bfloat16, like every other matrix operand of this precision.
 // DIM and VDIM are the PADDED sizes (32, 64 or 128): the real dim / vdim values (any multiple of 8) sit at the start of
 // the columns and the rest is zero; 16-wide steps that are all padding are skipped.  A bias table of up to kMmBiasMax
-// distances is staged (this head's column) in shared memory.
+// distances is staged (this head's column) in shared memory.  SIGM: sigmoid weights (no running maximum, no sum, no
+// rescaling of the accumulators).  SHARED: the values are the key rows, so ONE staged tile serves both products.
 constexpr int kMmRows = 64, kMmKeys = 64, kMmThreads = 128, kMmPad = 8, kMmStages = 2, kMmBiasMax = 4096;
 
 __device__ __forceinline__ float ma_tanh(float x) {        // 1 - 2 / (e^{2x} + 1), relative error ~1e-6
@@ -580,15 +675,17 @@ __device__ __forceinline__ float ma_tanh(float x) {        // 1 - 2 / (e^{2x} + 
     return 1.0f - __fdividef(2.0f, e + 1.0f);
 }
 
-template <int DIM, int VDIM>
+template <int DIM, int VDIM, bool SIGM, bool SHARED>
 __global__ void __launch_bounds__(kMmThreads) masked_attention_mma_kernel(const MaskAttnParams p) {
+    static_assert(!SHARED || DIM == VDIM, "values that are the keys have their size");
     constexpr int KS = DIM + kMmPad, VS = VDIM + kMmPad, NT = VDIM / 8, NST = kMmStages;
     extern __shared__ __align__(16) unsigned char mm_smem[];
     bf16_t* Qs = reinterpret_cast<bf16_t*>(mm_smem);         // [64][KS]
     bf16_t* Ks = Qs + kMmRows * KS;                           // [NST][64][KS]
-    bf16_t* Vs = Ks + NST * kMmKeys * KS;                     // [NST][64][VS]
+    bf16_t* Vs = SHARED ? Ks : Ks + NST * kMmKeys * KS;       // [NST][64][VS]
     float* Bs = reinterpret_cast<float*>(Vs + NST * kMmKeys * VS);   // [bias_len] (bias_kind 2, bias_len <= kMmBiasMax)
     __shared__ int key_ok[NST][kMmKeys];
+    __shared__ __align__(8) float key_sc[NST][kMmKeys];
 
     const int* tile = p.tiles + 4 * blockIdx.x;
     const int row0 = tile[0], ntok = tile[1], slot = tile[2], pos0 = tile[3];
@@ -625,7 +722,10 @@ __global__ void __launch_bounds__(kMmThreads) masked_attention_mma_kernel(const 
     auto load_tile = [&](int kt, int buf) {
         const int key = tid >> 1, q2 = tid & 1;
         const int64_t pr = pool_row(kt * kMmKeys + key);
-        if (q2 == 0) key_ok[buf][key] = pr >= 0;
+        if (q2 == 0) {
+            key_ok[buf][key] = pr >= 0;
+            if (p.key_scale) key_sc[buf][key] = pr >= 0 ? p.key_scale[pr] : 0.f;
+        }
         bf16_t* kdst = Ks + (buf * kMmKeys + key) * KS;
         const bf16_t* ksrc = kp + (pr >= 0 ? pr * dim : 0);
 #pragma unroll
@@ -634,6 +734,7 @@ __global__ void __launch_bounds__(kMmThreads) masked_attention_mma_kernel(const 
             const bool ok = pr >= 0 && cv < dim;
             cp_async_16(smem_u32(kdst + cv), ok ? ksrc + cv : kp, ok);
         }
+        if (SHARED) return;
         bf16_t* vdst = Vs + (buf * kMmKeys + key) * VS;
         const bf16_t* vsrc = vp + (pr >= 0 ? pr * vdim : 0);
 #pragma unroll
@@ -665,6 +766,7 @@ __global__ void __launch_bounds__(kMmThreads) masked_attention_mma_kernel(const 
     const int wlo = ma_first_key(p, pos0 + rbase), whi = pos0 + min(rbase + 15, ntok - 1);
     const float slope = p.bias_kind == 1 ? p.bias[head] : 0.f;
     const float hscale = p.head_scale ? p.head_scale[head] : 1.f;
+    const float hbias = p.head_bias ? p.head_bias[head] : 0.f;
     const float inv_cap = p.softcap > 0.f ? 1.0f / p.softcap : 0.f;
     constexpr float kLog2e = 1.4426950408889634f;
 
@@ -700,11 +802,13 @@ __global__ void __launch_bounds__(kMmThreads) masked_attention_mma_kernel(const 
         for (int t = 0; t < 8; ++t) {
             const int col = t * 8 + 2 * (lane & 3);
             const int2 okk = *reinterpret_cast<const int2*>(&key_ok[buf][col]);
+            const float2 ksc = p.key_scale ? *reinterpret_cast<const float2*>(&key_sc[buf][col]) : make_float2(1.f, 1.f);
 #pragma unroll
             for (int c = 0; c < 4; ++c) {
                 const int i = c >> 1, j = c0 + col + (c & 1);
                 const bool vis = ((c & 1) ? okk.y : okk.x) && j <= rpos[i] && (j >= rlo[i] || j < keep);
                 float v = s[t][c] * p.scale;
+                if (p.key_scale) v *= (c & 1) ? ksc.y : ksc.x;
                 if (p.head_scale) v *= hscale;
                 if (p.softcap > 0.f) v = p.softcap * ma_tanh(v * inv_cap);
                 if (p.bias_kind == 1) v -= slope * (float)(rpos[i] - j);
@@ -712,10 +816,15 @@ __global__ void __launch_bounds__(kMmThreads) masked_attention_mma_kernel(const 
                     const int dist = min(rpos[i] - j, p.bias_len - 1);
                     v += bias_smem ? Bs[dist] : p.bias[(int64_t)dist * p.heads + head];
                 }
-                s[t][c] = vis ? v * kLog2e : -INFINITY;
+                if (SIGM) {
+                    s[t][c] = vis ? __fdividef(1.0f, 1.0f + exp2f(-kLog2e * (v + hbias))) : 0.f;
+                    continue;
+                }
+                s[t][c] = vis ? (v + hbias) * kLog2e : -INFINITY;
                 mx[i] = fmaxf(mx[i], s[t][c]);
             }
         }
+        if (!SIGM) {
         float ref[2];
 #pragma unroll
         for (int i = 0; i < 2; ++i) {
@@ -739,6 +848,7 @@ __global__ void __launch_bounds__(kMmThreads) masked_attention_mma_kernel(const 
                 s[t][c] = exp2f(s[t][c] - ref[c >> 1]);
                 l[c >> 1] += s[t][c];
             }
+        }
         // ---- weighted sums
 #pragma unroll
         for (int kk = 0; kk < 4; ++kk) {
@@ -768,8 +878,8 @@ __global__ void __launch_bounds__(kMmThreads) masked_attention_mma_kernel(const 
         l[i] += __shfl_xor_sync(0xffffffffu, l[i], 2);
         const int r = rbase + (lane >> 2) + 8 * i;
         if (r >= ntok) continue;
-        float inv = 1.0f / l[i];
-        if (p.sink) {                                        // the running maximum is in the log2 domain
+        float inv = SIGM ? 1.0f : 1.0f / l[i];
+        if (!SIGM && p.sink) {                                        // the running maximum is in the log2 domain
             const float sk = p.sink[head] * kLog2e, mn = fmaxf(m[i], sk);
             const float corr = exp2f(m[i] - mn);
             inv = corr / (l[i] * corr + exp2f(sk - mn));
@@ -785,16 +895,22 @@ __global__ void __launch_bounds__(kMmThreads) masked_attention_mma_kernel(const 
                 u = ma_unturn(p, row0 + r, col, u0, v);
                 v = ma_unturn(p, row0 + r, col + 1, v, u0);
             }
+            if (p.gate) {
+                const int col = head * vdim + t * 8 + 2 * (lane & 3);
+                u *= ma_gate<bf16_t>(p, row0 + r, col);
+                v *= ma_gate<bf16_t>(p, row0 + r, col + 1);
+            }
             *reinterpret_cast<uint32_t*>(dst + t * 8) = pack_bf16x2(u, v);
         }
     }
 }
 
-template <int DIM, int VDIM>
+template <int DIM, int VDIM, bool SIGM, bool SHARED>
 static int mm_launch(const MaskAttnParams& p, int ntiles, cudaStream_t st) {
-    size_t smem = ((size_t)(kMmRows + kMmStages * kMmKeys) * (DIM + kMmPad) + (size_t)kMmStages * kMmKeys * (VDIM + kMmPad)) * sizeof(bf16_t);
+    size_t smem = ((size_t)(kMmRows + kMmStages * kMmKeys) * (DIM + kMmPad) +
+                   (SHARED ? 0 : (size_t)kMmStages * kMmKeys * (VDIM + kMmPad))) * sizeof(bf16_t);
     if (p.bias_kind == 2 && p.bias_len <= kMmBiasMax) smem += (size_t)p.bias_len * sizeof(float);
-    auto kern = masked_attention_mma_kernel<DIM, VDIM>;
+    auto kern = masked_attention_mma_kernel<DIM, VDIM, SIGM, SHARED>;
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
     dim3 grid((unsigned)ntiles, (unsigned)p.heads);
@@ -810,7 +926,13 @@ static int mm_dispatch(const MaskAttnParams& p, int ntiles, cudaStream_t st) {
     if (!mm_shape_ok(p.dim, p.vdim) || p.q_stride % 8 || p.q_off % 8) return PA_ERR_UNSUPPORTED;
     if ((uintptr_t)p.q % 16 || (uintptr_t)p.k_pool % 16 || (uintptr_t)p.v_pool % 16 || (uintptr_t)p.out % 4) return PA_ERR_UNSUPPORTED;
     const int dp = mm_padded(p.dim), vp = mm_padded(p.vdim);
-#define PA_MM_CASE(D, V) if (dp == D && vp == V) return mm_launch<D, V>(p, ntiles, st)
+    if (p.k_pool == p.v_pool) {
+#define PA_MM_CASE(D) if (dp == D) return p.sigm ? mm_launch<D, D, true, true>(p, ntiles, st) : mm_launch<D, D, false, true>(p, ntiles, st)
+        PA_MM_CASE(32); PA_MM_CASE(64); PA_MM_CASE(128);
+#undef PA_MM_CASE
+        return PA_ERR_UNSUPPORTED;
+    }
+#define PA_MM_CASE(D, V) if (dp == D && vp == V) return p.sigm ? mm_launch<D, V, true, false>(p, ntiles, st) : mm_launch<D, V, false, false>(p, ntiles, st)
     PA_MM_CASE(32, 32); PA_MM_CASE(32, 64); PA_MM_CASE(32, 128);
     PA_MM_CASE(64, 32); PA_MM_CASE(64, 64); PA_MM_CASE(64, 128);
     PA_MM_CASE(128, 32); PA_MM_CASE(128, 64); PA_MM_CASE(128, 128);
@@ -846,6 +968,21 @@ PA_API int pa_masked_attention_sink(const void* d_q, int64_t q_stride, int q_off
                                     float scale, float softcap, int mask_kind, int mask_size, int mask_keep, int bias_kind,
                                     const float* d_bias, int bias_len, const float* d_head_scale, const float* d_sink,
                                     const float* d_out_rot, void* d_out, int elem, int tile_kind, pa_stream_t stream) {
+    return pa_masked_attention_gated(d_q, q_stride, q_off, d_k_pool, d_v_pool, d_table, num_slots, num_kv_heads, num_tiles,
+                                     total_pages, tile_size, d_q_tiles, num_q_tiles, heads, dim, vdim, scale, softcap,
+                                     mask_kind, mask_size, mask_keep, bias_kind, d_bias, bias_len, d_head_scale, d_sink,
+                                     d_out_rot, nullptr, 0, nullptr, nullptr, 0, 0, d_out, elem, tile_kind, stream);
+}
+
+PA_API int pa_masked_attention_gated(const void* d_q, int64_t q_stride, int q_off, const void* d_k_pool, const void* d_v_pool,
+                                     const int32_t* d_table, int num_slots, int num_kv_heads, int num_tiles, int total_pages,
+                                     int tile_size, const int32_t* d_q_tiles, int num_q_tiles, int heads, int dim, int vdim,
+                                     float scale, float softcap, int mask_kind, int mask_size, int mask_keep, int bias_kind,
+                                     const float* d_bias, int bias_len, const float* d_head_scale, const float* d_sink,
+                                     const float* d_out_rot, const float* d_key_scale, int sigmoid_weights,
+                                     const float* d_head_bias, const void* d_gate, int64_t gate_stride, int gate_off,
+                                     void* d_out, int elem, int tile_kind, pa_stream_t stream) {
+    PA_CHECK_ARG((sigmoid_weights == 0 || sigmoid_weights == 1) && !(sigmoid_weights && d_sink) && (d_k_pool != d_v_pool || dim == vdim));
     PA_CHECK_ARG(mask_keep >= 0 && (mask_keep == 0 || mask_kind == 1) && (!d_out_rot || vdim % 2 == 0));
     PA_CHECK_ARG(d_q && d_k_pool && d_v_pool && d_table && d_q_tiles && d_out && num_q_tiles >= 0);
     PA_CHECK_ARG(num_slots > 0 && num_kv_heads > 0 && num_tiles > 0 && total_pages > 0 && tile_size > 0);
@@ -860,6 +997,8 @@ PA_API int pa_masked_attention_sink(const void* d_q, int64_t q_stride, int q_off
     p.softcap = softcap; p.mask_kind = mask_kind; p.mask_size = mask_size; p.bias_kind = bias_kind; p.bias = d_bias;
     p.bias_len = bias_len; p.out = d_out; p.head_rows = 0;
     p.head_scale = d_head_scale; p.sink = d_sink; p.mask_keep = mask_keep; p.out_rot = d_out_rot;
+    p.sigm = sigmoid_weights; p.key_scale = d_key_scale; p.head_bias = d_head_bias; p.gate = d_gate;
+    p.gate_stride = gate_stride; p.gate_off = gate_off;
     if (elem != 4 && elem != 2) return PA_ERR_UNSUPPORTED;
     if (tile_kind == 2) {       // on the tensor cores: tiles of up to pa_masked_attention_mma_tile_tokens tokens
         if (elem != 2) return PA_ERR_UNSUPPORTED;
@@ -891,6 +1030,23 @@ PA_API int pa_rope_kv_append(void* d_src, int64_t src_stride, int q_off, int k_o
                                rot_dims ? d_rope : nullptr, d_value_rope, static_cast<T*>(d_k_pool),
                                static_cast<T*>(d_v_pool), d_table, num_slots, num_tiles, total_pages, tile_size, d_row_slot,
                                d_row_pos, rows));
+    PA_RETURN_LAUNCH_STATUS();
+}
+
+PA_API int pa_qk_norm_kv_append(void* d_src, int64_t src_stride, int q_off, int k_off, int v_off, int heads, int kv_heads,
+                                int dim, int vdim, const float* d_q_gain, const float* d_k_gain, float eps, void* d_k_pool,
+                                void* d_v_pool, float* d_key_scale, const int32_t* d_table, int num_slots, int num_tiles,
+                                int total_pages, int tile_size, const int32_t* d_row_slot, const int32_t* d_row_pos,
+                                int rows, int elem, pa_stream_t stream) {
+    PA_CHECK_ARG(d_src && rows >= 0 && heads > 0 && kv_heads > 0 && dim > 0 && d_q_gain && (d_k_gain || d_key_scale));
+    PA_CHECK_ARG(d_k_pool && d_table && d_row_slot && d_row_pos && num_slots > 0 && num_tiles > 0 && total_pages > 0);
+    PA_CHECK_ARG(tile_size > 0 && d_v_pool != d_k_pool && (!d_v_pool || vdim > 0));
+    if (rows == 0) return PA_OK;
+    const int64_t threads = (int64_t)rows * (heads + kv_heads) * 32;
+    PA_DISPATCH_ELEM(elem, qk_norm_kv_append_kernel<T><<<(unsigned)((threads + 255) / 256), 256, 0, as_stream(stream)>>>(
+                               static_cast<T*>(d_src), src_stride, q_off, k_off, v_off, heads, kv_heads, dim, vdim, d_q_gain,
+                               d_k_gain, eps, static_cast<T*>(d_k_pool), static_cast<T*>(d_v_pool), d_key_scale, d_table,
+                               num_slots, num_tiles, total_pages, tile_size, d_row_slot, d_row_pos, rows));
     PA_RETURN_LAUNCH_STATUS();
 }
 

@@ -8,11 +8,13 @@
 //   decay_scan_kernel         S_t = a_t S_{t-1} + k_t (s_t v_t)^T,  o_t = S_t^T q_t + skip * v_t   per head, S is dim x vdim,
 //                             float, one slot per sequence.  The decay is a constant of the head (linear attention with
 //                             decay), or a_t = exp(-exp(A_log) dt_t) with dt_t = softplus(raw_t + bias) and s_t = dt_t
-//                             (selective state space); q / k may be shared by the heads of a group; q, k, v may pass silu
+//                             (selective state space); q / k may be shared by the heads of a group; q, k, v may pass silu;
+//                             q and k may be rotated (halves) over their first dimensions and k scaled, in float, as they
+//                             are staged
 //   decay_chunk_* kernels     the same recurrence for long portions as a three-pass chunked scan (fold every chunk from a
 //                             zero state, chain the chunks from the state slot, replay every chunk from its incoming state)
-//   gated_norm_kernel         RMS norm in equal groups of a float row with a per-channel weight and a gate from another
-//                             buffer: silu(gate) multiplied in BEFORE the norm, or sigmoid(gate) AFTER it
+//   gated_norm_kernel         RMS norm in equal groups of a float row with a per-channel weight (optional) and a gate from
+//                             another buffer: silu(gate) multiplied in BEFORE the norm, or sigmoid(gate) or silu(gate) AFTER
 //
 // States, decays and their logarithms, softplus, step sizes and the norms are float whatever the activation type.
 #include "seq_common.cuh"
@@ -101,6 +103,8 @@ struct DecayScanParams {
     int mode;
     int vec;                                          // every staged piece of q, k and v starts on a 16-byte boundary
     float* part;                                      // [items][heads][dim * vdim + 1]: state, then the chunk's total decay
+    const float* rope; int rot_dims;                  // [rows][rot_dims / 2][cos, sin]: pairs (i, i + rot_dims / 2) of q and k
+    float k_scale;                                    // multiplies k (constant decays)
 };
 
 constexpr int kDsTokens = 16;                         // tokens staged per step
@@ -222,7 +226,7 @@ __global__ void __launch_bounds__(kDsMaxThreads) decay_scan_kernel(const DecaySc
         }
         }
         if (threadIdx.x < nt) {
-            float a = hd, sc = 1.f;
+            float a = hd, sc = p.k_scale;              // the key's factor rides on its value: only k v^T is kept
             if (p.dt) {
                 const float raw = to_f32<T>(static_cast<const T*>(p.dt)[(int64_t)(row0 + t0 + threadIdx.x) * p.dt_stride + p.dt_off + h]);
                 sc = softplus_f32(raw + dtb);
@@ -232,6 +236,24 @@ __global__ void __launch_bounds__(kDsMaxThreads) decay_scan_kernel(const DecaySc
             Ss[threadIdx.x] = sc;
         }
         __syncthreads();
+        if (p.rope) {
+            const int half = p.rot_dims >> 1;
+            for (int idx = threadIdx.x; idx < nt * half; idx += blockDim.x) {
+                const int t = idx / half, i = idx % half;
+                const float2 cs = *reinterpret_cast<const float2*>(p.rope + ((int64_t)(row0 + t0 + t) * half + i) * 2);
+                float* kr = Ks + t * dpad + i;
+                const float ku = kr[0], kw = kr[half];
+                kr[0] = ku * cs.x - kw * cs.y;
+                kr[half] = kw * cs.x + ku * cs.y;
+                if (MODE != 1) {
+                    float* qr = Qs + t * dpad + i;
+                    const float qu = qr[0], qw = qr[half];
+                    qr[0] = qu * cs.x - qw * cs.y;
+                    qr[half] = qw * cs.x + qu * cs.y;
+                }
+            }
+            __syncthreads();
+        }
         for (int t = 0; t < nt; ++t) {
             const float a = As[t], sc = Ss[t];
             float x[CPT];
@@ -323,7 +345,8 @@ __global__ void __launch_bounds__(256) decay_chunk_chain_kernel(float* __restric
 }
 
 // ---- gated group norm ---------------------------------------------------------------------------------------------------
-// One warp per (row, group).  gate_mode 0: none; 1: y <- y * silu(gate) before the norm; 2: out <- norm(y) * sigmoid(gate).
+// One warp per (row, group).  gate_mode 0: none; 1: y <- y * silu(gate) before the norm; 2: out <- norm(y) * sigmoid(gate);
+// 3: out <- norm(y) * silu(gate).  weight may be null (ones).
 template <typename T>
 __global__ void __launch_bounds__(256) gated_norm_kernel(const float* __restrict__ y, int64_t rows, int inner, int groups,
                                                          const T* __restrict__ gate, int64_t gate_stride, int gate_off,
@@ -347,8 +370,10 @@ __global__ void __launch_bounds__(256) gated_norm_kernel(const float* __restrict
     for (int j = lane; j < gsz; j += 32) {
         float v = yr[j];
         if (gate_mode == 1) v *= silu_f32(to_f32<T>(gr[j]));
-        v = v * rn * weight[c0 + j];
+        v *= rn;
+        if (weight) v *= weight[c0 + j];
         if (gate_mode == 2) v *= sigmoid_f32(to_f32<T>(gr[j]));
+        if (gate_mode == 3) v *= silu_f32(to_f32<T>(gr[j]));
         out[r * inner + c0 + j] = from_f32<T>(v);
     }
 }
@@ -375,8 +400,10 @@ __global__ void __launch_bounds__(256) gated_norm_block_kernel(const float* __re
     for (int j = threadIdx.x; j < gsz; j += blockDim.x) {
         float v = yr[j];
         if (gate_mode == 1) v *= silu_f32(to_f32<T>(gr[j]));
-        v = v * rn * weight[c0 + j];
+        v *= rn;
+        if (weight) v *= weight[c0 + j];
         if (gate_mode == 2) v *= sigmoid_f32(to_f32<T>(gr[j]));
+        if (gate_mode == 3) v *= silu_f32(to_f32<T>(gr[j]));
         out[r * inner + c0 + j] = from_f32<T>(v);
     }
 }
@@ -473,9 +500,23 @@ PA_API int pa_decay_scan(const void* d_q, int64_t q_stride, int q_off, const voi
                          const int32_t* d_items, int num_items, const int32_t* d_seq_chunk0, const int32_t* d_seq_nchunks,
                          const int32_t* d_seq_slot, int num_seqs, int chunked, void* d_workspace, size_t workspace_bytes,
                          int elem, pa_stream_t stream) {
+    return pa_decay_scan_rotated(d_q, q_stride, q_off, d_k, k_stride, k_off, d_v, v_stride, v_off, heads, groups, dim, vdim, act,
+                                 d_decay, d_dt, dt_stride, dt_off, d_dt_bias, d_a_log, d_skip, nullptr, 0, 1.0f, d_state, d_out,
+                                 out_stride, d_items, num_items, d_seq_chunk0, d_seq_nchunks, d_seq_slot, num_seqs, chunked,
+                                 d_workspace, workspace_bytes, elem, stream);
+}
+
+PA_API int pa_decay_scan_rotated(const void* d_q, int64_t q_stride, int q_off, const void* d_k, int64_t k_stride, int k_off,
+                         const void* d_v, int64_t v_stride, int v_off, int heads, int groups, int dim, int vdim, int act,
+                         const float* d_decay, const void* d_dt, int64_t dt_stride, int dt_off, const float* d_dt_bias,
+                         const float* d_a_log, const float* d_skip, const float* d_rope, int rot_dims, float k_scale, float* d_state, float* d_out, int64_t out_stride,
+                         const int32_t* d_items, int num_items, const int32_t* d_seq_chunk0, const int32_t* d_seq_nchunks,
+                         const int32_t* d_seq_slot, int num_seqs, int chunked, void* d_workspace, size_t workspace_bytes,
+                         int elem, pa_stream_t stream) {
     PA_CHECK_ARG(d_q && d_k && d_v && d_state && d_out && d_items && num_items >= 0);
     PA_CHECK_ARG(heads > 0 && groups > 0 && heads % groups == 0 && dim > 0 && vdim > 0);
     PA_CHECK_ARG(d_dt ? (d_dt_bias && d_a_log) : d_decay != nullptr);
+    PA_CHECK_ARG(rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= dim && (rot_dims == 0 || d_rope) && (!d_dt || k_scale == 1.0f));
     if (num_items == 0) return PA_OK;
     if (elem != 4 && elem != 2) return PA_ERR_UNSUPPORTED;
     DecayScanParams p;
@@ -483,7 +524,7 @@ PA_API int pa_decay_scan(const void* d_q, int64_t q_stride, int q_off, const voi
     p.v = d_v; p.v_stride = v_stride; p.v_off = v_off; p.heads = heads; p.groups = groups; p.dim = dim; p.vdim = vdim;
     p.act = act; p.decay = d_decay; p.dt = d_dt; p.dt_stride = dt_stride; p.dt_off = dt_off; p.dt_bias = d_dt_bias;
     p.a_log = d_a_log; p.skip = d_skip; p.state = d_state; p.out = d_out; p.out_stride = out_stride; p.items = d_items;
-    p.part = static_cast<float*>(d_workspace);
+    p.part = static_cast<float*>(d_workspace); p.rope = rot_dims ? d_rope : nullptr; p.rot_dims = rot_dims; p.k_scale = k_scale;
     cudaStream_t st = as_stream(stream);
 #define PA_DS(MODE)                                                                                \
     do {                                                                                           \
@@ -509,8 +550,8 @@ PA_API int pa_decay_scan(const void* d_q, int64_t q_stride, int q_off, const voi
 PA_API int pa_gated_rms_norm(const float* d_y, int64_t rows, int inner, int groups, const void* d_gate, int64_t gate_stride,
                              int gate_off, int gate_mode, const float* d_weight, float eps, void* d_out, int elem,
                              pa_stream_t stream) {
-    PA_CHECK_ARG(d_y && d_weight && d_out && rows >= 0 && inner > 0 && groups > 0 && inner % groups == 0);
-    PA_CHECK_ARG(gate_mode >= 0 && gate_mode <= 2 && (gate_mode == 0 || d_gate));
+    PA_CHECK_ARG(d_y && d_out && rows >= 0 && inner > 0 && groups > 0 && inner % groups == 0);
+    PA_CHECK_ARG(gate_mode >= 0 && gate_mode <= 3 && (gate_mode == 0 || d_gate));
     if (rows == 0) return PA_OK;
     if (inner / groups >= 512 && rows * groups < (1 << 30)) {
         PA_DISPATCH_ELEM(elem, gated_norm_block_kernel<T><<<(unsigned)(rows * groups), 256, 0, as_stream(stream)>>>(

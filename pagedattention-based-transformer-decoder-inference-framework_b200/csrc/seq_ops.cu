@@ -16,6 +16,9 @@
 //   residual_add_prenorm_kernel  x += a * y + b * y2 + sum_k w_k * routed expert rows + shared + bias, then the NEXT
 //                             sublayer's operand h = x / rms(x) * gain in the activation type (pre-norm wiring: the
 //                             residual add of one sublayer fused with the norm in front of the next)
+//   streams_add_norm_kernel   the residual kept as several streams: every stream becomes a mix of the old ones plus its
+//                             share of the sublayer's output, and the next sublayer's operand is the norm of a weighted sum
+//                             of the new streams
 //   concat_rows_kernel        [x | x0] of two float row sets in the activation type (input of a looped block)
 //   residual_add_norm2_kernel  the parallel wiring with two norms: x += the sublayers' outputs (routed experts by weight,
 //                             identity experts = the feed-forward's own input row), then BOTH operands of the next layer,
@@ -447,6 +450,104 @@ __global__ void __launch_bounds__(256) residual_add_norm2_kernel(float* __restri
 }
 
 // One CTA per row of `ff` values: the mean squares of z, z^2 and z^3 in one pass, then the weighted sum.
+// One CTA per row of a residual kept as `streams` float rows.  With x_s the old streams (src: [rows][src_streams][width];
+// src_streams == 1: all of them are the one row there):
+//     x'_t = sum_s mix[s][t] x_s + out[t] y      (mix == null: x'_t = x_t, nothing is added)
+//     u    = sum_t in[t] x'_t                    (in == null: ones)
+// x' goes to dst ([rows][streams][width], may be src; null: not kept), u to u_out (float, optional), and
+// next = u / rms(u) * gain in the activation type (optional).  row_ids != null: row r of the outputs is batch row row_ids[r].
+constexpr int kMaxStreams = 16;
+
+template <typename T, int MAXS, int VEC>
+__global__ void __launch_bounds__(256) streams_add_norm_kernel(const float* src, int src_streams, float* dst, int streams,
+                                                               int width, const T* __restrict__ y,
+                                                               const float* __restrict__ mix, const float* __restrict__ out_w,
+                                                               const float* __restrict__ in_w, float eps,
+                                                               const float* __restrict__ gain, float* __restrict__ u_out,
+                                                               T* __restrict__ next, const int32_t* __restrict__ row_ids) {
+    extern __shared__ __align__(16) float st_row[];    // [width]
+    __shared__ float sm[32], ms[MAXS * MAXS], os[MAXS], is[MAXS];
+    const int S = MAXS <= 4 ? MAXS : streams;          // up to four streams the count is the template's
+    const int64_t r = blockIdx.x, b = row_ids ? row_ids[r] : r;
+    for (int i = threadIdx.x; i < S * S; i += blockDim.x) ms[i] = mix ? mix[i] : (i / S == i % S ? 1.f : 0.f);
+    for (int i = threadIdx.x; i < S; i += blockDim.x) {
+        os[i] = mix && out_w ? out_w[i] : 0.f;
+        is[i] = in_w ? in_w[i] : 1.f;
+    }
+    __syncthreads();
+    const float* xs = src + b * src_streams * width;
+    float* xd = dst ? dst + b * S * width : nullptr;
+    float ss = 0.f;
+    for (int j = threadIdx.x * VEC; j < width; j += blockDim.x * VEC) {
+        float x[MAXS][VEC], yv[VEC], u[VEC];
+#pragma unroll
+        for (int s = 0; s < MAXS; ++s) {
+            if (s >= S) break;
+            const float* p = xs + (src_streams == 1 ? 0 : (int64_t)s * width) + j;
+            if (VEC == 4) {
+                const float4 v = *reinterpret_cast<const float4*>(p);
+                x[s][0] = v.x; x[s][1 % VEC] = v.y; x[s][2 % VEC] = v.z; x[s][3 % VEC] = v.w;
+            } else {
+                x[s][0] = p[0];
+            }
+        }
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) { yv[i] = 0.f; u[i] = 0.f; }
+        if (y) {
+            const T* p = y + b * width + j;
+            if (VEC == 4 && sizeof(T) == 2) {
+                const uint2 v = *reinterpret_cast<const uint2*>(p);
+                yv[0] = __uint_as_float(v.x << 16); yv[1 % VEC] = __uint_as_float(v.x & 0xffff0000u);
+                yv[2 % VEC] = __uint_as_float(v.y << 16); yv[3 % VEC] = __uint_as_float(v.y & 0xffff0000u);
+            } else {
+#pragma unroll
+                for (int i = 0; i < VEC; ++i) yv[i] = to_f32<T>(p[i]);
+            }
+        }
+#pragma unroll
+        for (int t = 0; t < MAXS; ++t) {
+            if (t >= S) break;
+            float v[VEC];
+            const float o = os[t], a = is[t];
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) v[i] = o * yv[i];
+#pragma unroll
+            for (int s = 0; s < MAXS; ++s) {
+                if (s >= S) break;
+                const float m = ms[s * S + t];
+#pragma unroll
+                for (int i = 0; i < VEC; ++i) v[i] = fmaf(m, x[s][i], v[i]);
+            }
+            if (xd) {
+                if (VEC == 4) *reinterpret_cast<float4*>(xd + (int64_t)t * width + j) = make_float4(v[0], v[1 % VEC], v[2 % VEC], v[3 % VEC]);
+                else xd[(int64_t)t * width + j] = v[0];
+            }
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) u[i] = fmaf(a, v[i], u[i]);
+        }
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) {
+            st_row[j + i] = u[i];
+            ss = fmaf(u[i], u[i], ss);
+            if (u_out) u_out[r * width + j + i] = u[i];
+        }
+    }
+    if (!next) return;
+    ss = block_sum(ss, sm);
+    const float rn = 1.0f / sqrtf(ss / (float)width + eps);
+    for (int j = threadIdx.x * VEC; j < width; j += blockDim.x * VEC) {     // a thread reads back its own columns
+        float f[VEC];
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) f[i] = st_row[j + i] * rn * gain[j + i];
+        if (VEC == 4 && sizeof(T) == 2) {
+            *reinterpret_cast<uint2*>(next + r * width + j) = make_uint2(pack_bf16x2(f[0], f[1 % VEC]), pack_bf16x2(f[2 % VEC], f[3 % VEC]));
+        } else {
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) next[r * width + j + i] = from_f32<T>(f[i]);
+        }
+    }
+}
+
 template <typename T>
 __global__ void __launch_bounds__(256) poly_norm_kernel(const T* __restrict__ z, int ff, const float* __restrict__ coef,
                                                         float eps, T* __restrict__ out) {
@@ -664,6 +765,36 @@ PA_API int pa_residual_add_norm2(float* d_x, int64_t rows, int width, const void
                                d_x, width, static_cast<const T*>(d_y), static_cast<const T*>(d_y2), d_routed, d_sel_w,
                                d_sel_id, top, experts, static_cast<const T*>(d_ident), eps, d_gain1,
                                static_cast<T*>(d_next1), d_gain2, static_cast<T*>(d_next2)));
+    PA_RETURN_LAUNCH_STATUS();
+}
+
+PA_API int pa_streams_add_norm(const float* d_src, int src_streams, float* d_dst, int64_t rows, int streams, int width,
+                               const void* d_y, const float* d_mix, const float* d_out_w, const float* d_in_w, float eps,
+                               const float* d_gain, float* d_u, void* d_next, const int32_t* d_row_ids, int elem,
+                               pa_stream_t stream) {
+    PA_CHECK_ARG(d_src && rows >= 0 && width > 0 && streams > 0 && (src_streams == 1 || src_streams == streams));
+    PA_CHECK_ARG((d_y != nullptr) == (d_mix != nullptr) && (!d_y || d_out_w) && (!d_next || d_gain) && !(d_row_ids && d_dst));
+    PA_CHECK_ARG(!d_dst || d_dst != d_src || src_streams == streams);
+    if (rows == 0) return PA_OK;
+    const size_t smem = (size_t)width * sizeof(float);
+    if (smem > 46 * 1024 || streams > kMaxStreams) return PA_ERR_UNSUPPORTED;
+    auto al = [](const void* p, int n) { return (uintptr_t)p % n == 0; };
+    const bool vec = width % 4 == 0 && al(d_src, 16) && al(d_dst, 16) && al(d_y, elem == 2 ? 8 : 16) && al(d_next, elem == 2 ? 8 : 16);
+#define PA_STREAMS(MAXS, VEC)                                                                                             \
+    PA_DISPATCH_ELEM(elem, streams_add_norm_kernel<T, MAXS, VEC><<<(unsigned)rows, 256, smem, as_stream(stream)>>>(       \
+                               d_src, src_streams, d_dst, streams, width, static_cast<const T*>(d_y), d_mix, d_out_w,     \
+                               d_in_w, eps, d_gain, d_u, static_cast<T*>(d_next), d_row_ids))
+#define PA_STREAMS_CASE(MAXS) if (vec) PA_STREAMS(MAXS, 4); else PA_STREAMS(MAXS, 1)
+    switch (streams <= 4 ? streams : streams <= 8 ? 8 : 16) {
+        case 1: PA_STREAMS_CASE(1); break;
+        case 2: PA_STREAMS_CASE(2); break;
+        case 3: PA_STREAMS_CASE(3); break;
+        case 4: PA_STREAMS_CASE(4); break;
+        case 8: PA_STREAMS_CASE(8); break;
+        default: PA_STREAMS_CASE(16); break;
+    }
+#undef PA_STREAMS_CASE
+#undef PA_STREAMS
     PA_RETURN_LAUNCH_STATUS();
 }
 

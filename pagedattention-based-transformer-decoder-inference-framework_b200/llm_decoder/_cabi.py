@@ -172,6 +172,19 @@ _SIGS = {
     "pa_logit_softcap": ([_vp, _i64, _f32, _f32, _vp], _i32),
     "pa_router_topk_biased": ([_vp, _vp, _vp, _vp, _i32, _i32, _i32, _i32, _i32, _i32, _i32, _i32, _vp, _vp, _vp, _vp, _i32,
                                _vp], _i32),
+    # sigmoid weights / keys as values / query-key norm / fused output gate; rotated retention; residual streams
+    "pa_masked_attention_gated": ([_vp, _i64, _i32, _vp, _vp, _vp, _i32, _i32, _i32, _i32, _i32, _vp, _i32, _i32, _i32, _i32,
+                                   _f32, _f32, _i32, _i32, _i32, _i32, _vp, _i32, _vp, _vp, _vp, _vp, _i32, _vp, _vp, _i64, _i32,
+                                   _vp, _i32, _i32, _vp], _i32),
+    "pa_qk_norm_kv_append": ([_vp, _i64, _i32, _i32, _i32, _i32, _i32, _i32, _i32, _vp, _vp, _f32, _vp, _vp, _vp, _vp, _i32,
+                              _i32, _i32, _i32, _vp, _vp, _i32, _i32, _vp], _i32),
+    "pa_decay_scan_rotated": ([_vp, _i64, _i32, _vp, _i64, _i32, _vp, _i64, _i32, _i32, _i32, _i32, _i32, _i32, _vp, _vp, _i64,
+                               _i32, _vp, _vp, _vp, _vp, _i32, _f32, _vp, _vp, _i64, _vp, _i32, _vp, _vp, _vp, _i32, _i32, _vp,
+                               _sz, _i32, _vp], _i32),
+    "pa_rope_rows_paired": ([_vp, _i64, _i32, _i32, _i32, _i32, _vp, _i32, _i32, _i32, _vp], _i32),
+    "pa_latent_norm_append": ([_vp, _vp, _i32, _i32, _i32, _i32, _i32, _i32, _i32, _i32, _vp, _i64, _i32, _vp, _f32, _vp, _i32,
+                               _i32, _vp, _vp, _i64, _vp, _vp, _i32, _i32, _vp], _i32),
+    "pa_streams_add_norm": ([_vp, _i32, _vp, _i64, _i32, _i32, _vp, _vp, _vp, _vp, _f32, _vp, _vp, _vp, _vp, _i32, _vp], _i32),
     "pa_causal_conv": ([_vp, _i64, _i32, _i32, _i32, _vp, _vp, _i32, _vp, _vp, _i32, _vp, _i64, _i32, _vp], _i32),
 }
 

@@ -214,6 +214,9 @@ class DiffAttentionMixer:
         return c.model._linear(out, self.w_o)
 
 
+ROPE_PAIRING = {"neighbours": 0, "halves": 1}
+
+
 def latent_key_splits(ctas, longest, sms):
     """Too few CTAs for the chip over a long context: cut the keys into parts (at least 256 keys each), as many as still
     make ONE wave of CTAs -- the kernels hold most of an SM's shared memory, so a second, partial wave costs a whole one."""
@@ -225,10 +228,13 @@ def latent_key_splits(ctas, longest, sms):
 class LatentAttentionMixer:
     """Attention through a low-rank latent over a paged pool with ONE row per token (KVTileCache with one key/value head
     and no value pool: row = [c | kr]).  The per-head key and value maps are applied on the query side and after the
-    weighted sum (pa_head_linear), so a step reads kv_rank + rot_dim values per cached token whatever the head count."""
+    weighted sum (pa_head_linear), so a step reads kv_rank + rot_dim values per cached token whatever the head count.
+    A design picks the pairs of the rotation (pairing 'neighbours': (2i, 2i + 1), or 'halves': (i, i + dims / 2)) and
+    whether every head's output is gated by sigmoid(W_g h) (head_gate)."""
     kind = "latent_attention"
 
-    def __init__(self, model, prefix, cfg, W):
+    def __init__(self, model, prefix, cfg, W, pairing="neighbours", head_gate=True):
+        self.pairing, self.head_gate = ROPE_PAIRING[pairing], bool(head_gate)
         H, self.dim, self.rot_dim, self.vdim = int(cfg["heads"]), int(cfg["dim"]), int(cfg["rot_dim"]), int(cfg["vdim"])
         self.heads, self.kv_rank, self.q_rank = H, int(cfg["kv_rank"]), int(cfg["q_rank"])
         rot = cfg.get("rot") or {}
@@ -241,11 +247,12 @@ class LatentAttentionMixer:
         qd, kd = self.dim + self.rot_dim, self.kv_rank + self.rot_dim
         self.qd, self.kd = qd, kd
         for name, shape in (("dq", (self.q_rank, model.width)), ("uq", (H * qd, self.q_rank)), ("uk", (H * self.dim, self.kv_rank)),
-                            ("uv", (H * self.vdim, self.kv_rank)), ("g", (H, model.width)), ("o", (model.width, H * self.vdim))):
+                            ("uv", (H * self.vdim, self.kv_rank)), ("o", (model.width, H * self.vdim))) + (
+                                (("g", (H, model.width)),) if self.head_gate else ()):
             if tuple(W[prefix + name].shape) != shape:
                 raise ValueError(f"{prefix}{name}: shape {tuple(W[prefix + name].shape)} does not match the config {shape}")
-        # one product for everything that reads the layer's input: [dq | dkv (own pool only) | g]
-        parts = [W[prefix + "dq"]] + ([W[prefix + "dkv"]] if self.own_kv else []) + [W[prefix + "g"]]
+        # one product for everything that reads the layer's input: [dq | dkv (own pool only) | g (gated only)]
+        parts = ([W[prefix + "dq"]] + ([W[prefix + "dkv"]] if self.own_kv else []) + ([W[prefix + "g"]] if self.head_gate else []))
         self.w_in = model._weight(torch.cat(parts, 0))
         self.c_off = self.q_rank
         self.g_off = self.q_rank + (kd if self.own_kv else 0)
@@ -258,13 +265,14 @@ class LatentAttentionMixer:
             if tuple(W[prefix + "dkv"].shape) != (kd, model.width):
                 raise ValueError(f"{prefix}dkv: shape does not match kv_rank + rot_dim")
             self.dkv_gain = model._f32(W[prefix + "dkv.norm"])
-            self.kv = model.states.add_kv_layer(1, kd, 0, _KV[model.act_dtype])
+            self.alloc_state(model)
         else:
             j = int(self.kv_from)
             src = model.layers[j].mixer if 0 <= j < len(model.layers) else None
             if not isinstance(src, LatentAttentionMixer) or not src.own_kv:
                 raise ValueError(f"{prefix}: kv_from must name an earlier latent-attention layer with a pool of its own")
-            if (src.kv_rank, src.rot_dim, src.rot_dims, src.rot_base) != (self.kv_rank, self.rot_dim, self.rot_dims, self.rot_base):
+            if (src.kv_rank, src.rot_dim, src.rot_dims, src.rot_base, src.pairing) != (self.kv_rank, self.rot_dim, self.rot_dims,
+                                                                                       self.rot_base, self.pairing):
                 raise ValueError(f"{prefix}: kv_rank, rot_dim and rotation must equal those of layer {j}")
             self.kv = src.kv
         self.tile_tokens = model._lib.pa_latent_attention_tile_tokens(H)
@@ -273,14 +281,26 @@ class LatentAttentionMixer:
         if self.dim % 8 == 0 and qd % 8 == 0:
             self.mma_tokens = model._lib.pa_latent_attention_mma_tile_tokens(H, self.kv_rank, self.rot_dim, _ELEM[model.act_dtype])
 
-    def _head_linear(self, c, x, x_rs, x_hs, w, K, N):
-        """out[h, r, :] = x[r, h, :K] . w[h] for every head: [H, R, N] (row stride N, head stride R * N).  bfloat16: the
-        vendor's batched product on the strided view; float32: the IEEE FMA kernel."""
+    def alloc_state(self, model):
+        self.kv = model.states.add_kv_layer(1, self.kd, 0, _KV[model.act_dtype])
+
+    def new_pass(self, model):
+        if not self.own_kv:
+            raise ValueError("a layer that borrows keys and values cannot run in a looped block")
+        m = copy.copy(self)
+        m.alloc_state(model)
+        return m
+
+    def _head_linear(self, c, x, x_rs, x_hs, w, K, N, by_row=False):
+        """x[r, h, :K] . w[h] for every head: [H, R, N] (row stride N, head stride R * N), or by_row [R, H, N].  bfloat16:
+        the vendor's batched product on the strided views; float32: the IEEE FMA kernel."""
         H, R = self.heads, c.R
+        out = c.empty(R, H, N) if by_row else c.empty(H, R, N)
         if c.elem == 2:
-            return torch.bmm(torch.as_strided(x, (H, R, K), (x_hs, x_rs, 1)), w)
-        out = c.empty(H, R, N)
-        _chk(c.lib.pa_head_linear(x.data_ptr(), x_rs, x_hs, w.data_ptr(), H, K, N, R, out.data_ptr(), N, R * N, c.elem,
+            torch.bmm(torch.as_strided(x, (H, R, K), (x_hs, x_rs, 1)), w, out=out.transpose(0, 1) if by_row else out)
+            return out
+        o_rs, o_hs = (H * N, N) if by_row else (N, R * N)
+        _chk(c.lib.pa_head_linear(x.data_ptr(), x_rs, x_hs, w.data_ptr(), H, K, N, R, out.data_ptr(), o_rs, o_hs, c.elem,
                                   _cabi.stream()), "pa_head_linear")
         return out
 
@@ -315,20 +335,23 @@ class LatentAttentionMixer:
         b, lib, kv, s, R, H = c.batch, c.lib, self.kv, _cabi.stream(), c.R, self.heads
         proj = c.model._linear(h, self.w_in)
         cq = c.empty(R, self.q_rank)
-        _chk(lib.pa_rms_norm_rows(proj.data_ptr(), proj.stride(0), 0, self.q_rank, c.model.eps, self.dq_gain.data_ptr(),
-                                  cq.data_ptr(), self.q_rank, R, c.elem, s), "pa_rms_norm_rows")
-        q = c.model._linear(cq, self.w_uq)
         rope = c.rope_table(self.rot_dims, self.rot_base)
-        _chk(lib.pa_rope_rows(q.data_ptr(), q.stride(0), self.dim, self.qd, H, self.rot_dims, _cabi.ptr(rope), R, c.elem, s),
-             "pa_rope_rows")
         pt = kv.page_table_
         table = pt.device_data()
-        if self.own_kv:
-            _chk(lib.pa_latent_kv_append(kv.key_buffer_.data_ptr(), table.data_ptr(), pt.num_beams_, pt.num_tiles_,
-                                         kv.total_pages_, kv.tile_size_, self.kv_rank, self.rot_dim, self.rot_dims,
-                                         proj.data_ptr(), proj.stride(0), self.c_off, self.dkv_gain.data_ptr(), c.model.eps,
-                                         _cabi.ptr(rope), b.row_slot.data_ptr(), b.row_pos.data_ptr(), R, c.elem, s),
-                 "pa_latent_kv_append")
+        if self.own_kv:     # the norm of the query latent and the new pool rows: one launch
+            _chk(lib.pa_latent_norm_append(kv.key_buffer_.data_ptr(), table.data_ptr(), pt.num_beams_, pt.num_tiles_,
+                                           kv.total_pages_, kv.tile_size_, self.kv_rank, self.rot_dim, self.rot_dims,
+                                           self.pairing, proj.data_ptr(), proj.stride(0), self.c_off,
+                                           self.dkv_gain.data_ptr(), c.model.eps, _cabi.ptr(rope), 0, self.q_rank,
+                                           self.dq_gain.data_ptr(), cq.data_ptr(), self.q_rank, b.row_slot.data_ptr(),
+                                           b.row_pos.data_ptr(), R, c.elem, s), "pa_latent_norm_append")
+        else:
+            _chk(lib.pa_rms_norm_rows(proj.data_ptr(), proj.stride(0), 0, self.q_rank, c.model.eps, self.dq_gain.data_ptr(),
+                                      cq.data_ptr(), self.q_rank, R, c.elem, s), "pa_rms_norm_rows")
+        q = c.model._linear(cq, self.w_uq)
+        if self.rot_dims:
+            _chk(lib.pa_rope_rows_paired(q.data_ptr(), q.stride(0), self.dim, self.qd, H, self.rot_dims, _cabi.ptr(rope),
+                                         self.pairing, R, c.elem, s), "pa_rope_rows_paired")
         kvr = self.kv_rank
         ql = self._head_linear(c, q, q.stride(0), self.qd, self.w_uk, self.dim, kvr)          # [H, R, kv_rank]
         lat = c.empty(H, R, kvr)
@@ -336,6 +359,9 @@ class LatentAttentionMixer:
             self.mma_tokens = 0         # a stride or an alignment the tensor-core kernel does not take: the float kernel
         if self.mma_tokens == 0:
             self._attend(c, q, ql, lat, False)
+        if not self.head_gate:
+            ov = self._head_linear(c, lat, kvr, R * kvr, self.w_uv, kvr, self.vdim, by_row=True)
+            return c.model._linear(ov.view(R, H * self.vdim), self.w_o)
         ov = self._head_linear(c, lat, kvr, R * kvr, self.w_uv, kvr, self.vdim)               # [H, R, vdim]
         og = c.empty(R, H * self.vdim)
         _chk(lib.pa_head_gate(ov.data_ptr(), self.vdim, R * self.vdim, proj.data_ptr() + self.g_off * c.elem, proj.stride(0),
@@ -358,7 +384,7 @@ def log_distance_bucket(n, buckets, far):
 
 
 class MaskedAttention:
-    """Softmax attention with grouped key/value heads over a paged pool of its own; the design picks the visibility rule
+    """Softmax (or sigmoid) attention with grouped key/value heads over a paged pool of its own; the design picks the visibility rule
     (`mask`: 'causal', 'window' or 'chunk' of cfg mask.size; a window also keeps the first cfg mask.keep_first positions),
     the distance bias (`bias`: None, 'slope' -- minus 2^(-slope_exp (h + 1) / heads) per step of distance -- or 'bucket' --
     a learned table '<prefix>rel' [buckets, heads] over log_distance_bucket(distance, buckets, cfg bias_max)), whether cfg
@@ -373,13 +399,22 @@ class MaskedAttention:
       head_temp    a learned factor per query head on the scaled dot products ('<prefix>temp')
       sink         'learned': a logit per head ('<prefix>sink') in the softmax denominator, without key or value;
                    'zero': the same with logit 0 (one added to the denominator)
+      qk_norm      every query and key head divided by its root mean square, times '<prefix>q.norm' / '<prefix>k.norm' [dim]
+      values       'own', or 'keys': there is no value projection, the values are the keys before their norm -- the pool
+                   holds ONE row per key (as projected) and its inverse root mean square beside it; the norm's gain goes
+                   to the query side
+      weights      'softmax', or 'sigmoid': sigmoid(score) per visible key, nothing divides the sum
+      head_bias    a learned number per query head added to the score ('<prefix>pb')
+      gate         the heads' outputs times sigmoid(W_g h), element by element ('<prefix>g', part of the input product),
+                   applied inside the attention kernels
 
     A layer whose cfg has `kv_from: j` owns no key / value projections (nor their convolutions): it reads the pool of
     layer j (keys and values as cached there) with its own queries.  The mixer reads its q | k | v from a projection
     buffer at a column offset, so a mixer can fuse its input product with others."""
 
     def __init__(self, model, prefix, cfg, W, mask="causal", bias=None, softcap=False, slope_exp=8.0, proj_bias=True,
-                 conv=False, rot=False, rot_values=False, head_temp=False, sink=None):
+                 conv=False, rot=False, rot_values=False, head_temp=False, sink=None, qk_norm=False, values="own",
+                 weights="softmax", head_bias=False, gate=False):
         self.heads, self.kv_heads = int(cfg["heads"]), int(cfg["kv_heads"])
         self.dim, self.vdim = int(cfg["dim"]), int(cfg["vdim"])
         if self.heads % self.kv_heads:
@@ -392,7 +427,19 @@ class MaskedAttention:
         self.kv_from = cfg.get("kv_from")
         self.own_kv = self.kv_from is None
         H = self.heads
-        shapes = (("q", H * self.dim),) + ((("k", self.kv_heads * self.dim), ("v", self.kv_heads * self.vdim)) if self.own_kv else ())
+        self.qk_norm, self.keys_as_values = bool(qk_norm), values == "keys"
+        if values not in ("own", "keys") or weights not in ("softmax", "sigmoid"):
+            raise ValueError(f"unknown values {values!r} or weights {weights!r}")
+        self.sigmoid = 1 if weights == "sigmoid" else 0
+        if self.keys_as_values and (self.dim != self.vdim or not self.qk_norm):
+            raise ValueError(f"{prefix}: values that are the keys need vdim = dim and the query / key norm")
+        if self.qk_norm and (rot or rot_values or not self.own_kv):
+            raise ValueError(f"{prefix}: the query / key norm is served without rotation and on a pool of the layer's own")
+        if self.sigmoid and sink is not None:
+            raise ValueError(f"{prefix}: sigmoid weights have no denominator for a sink")
+        shapes = (("q", H * self.dim),)
+        if self.own_kv:
+            shapes += (("k", self.kv_heads * self.dim),) + ((("v", self.kv_heads * self.vdim),) if not self.keys_as_values else ())
         for name, rows in shapes:
             if tuple(W[prefix + name].shape) != (rows, model.width) or (proj_bias and tuple(W[prefix + name + ".b"].shape) != (rows,)):
                 raise ValueError(f"{prefix}{name}: shape does not match the config")
@@ -401,7 +448,26 @@ class MaskedAttention:
         self.in_weight = torch.cat([W[prefix + n] for n, _ in shapes], 0)
         self.in_bias = torch.cat([W[prefix + n + ".b"] for n, _ in shapes], 0) if proj_bias else None
         self.q_cols, self.k_cols = H * self.dim, self.kv_heads * self.dim
+        self.qkv_cols = int(self.in_weight.shape[0])
+        self.gate = bool(gate)
+        if self.gate:       # the gate's columns follow q | k | v
+            if tuple(W[prefix + "g"].shape) != (H * self.vdim, model.width) or (proj_bias and tuple(W[prefix + "g.b"].shape) != (H * self.vdim,)):
+                raise ValueError(f"{prefix}g: shape does not match the config")
+            self.in_weight = torch.cat([self.in_weight, W[prefix + "g"]], 0)
+            if proj_bias:
+                self.in_bias = torch.cat([self.in_bias, W[prefix + "g.b"]], 0)
         self.in_cols = int(self.in_weight.shape[0])
+        self.q_gain = self.k_gain = self.head_bias = None
+        if self.qk_norm:
+            for n in ("q.norm", "k.norm"):
+                if tuple(W[prefix + n].shape) != (self.dim,):
+                    raise ValueError(f"{prefix}{n}: one number per head dimension expected")
+            qg, kg = W[prefix + "q.norm"].to(torch.float32), W[prefix + "k.norm"].to(torch.float32)
+            self.q_gain, self.k_gain = model._f32(qg * kg if self.keys_as_values else qg), model._f32(kg)
+        if head_bias:
+            if tuple(W[prefix + "pb"].shape) != (H,):
+                raise ValueError(f"{prefix}pb: one number per head expected")
+            self.head_bias = model._f32(W[prefix + "pb"])
         self.w_o, self.b_o = model._weight(W[prefix + "o"]), model._bias(W[prefix + "o.b"]) if proj_bias else None
         self.taps, self.conv_w = 0, None
         if conv:
@@ -471,12 +537,13 @@ class MaskedAttention:
 
     def alloc_state(self, model):
         if self.own_kv:
-            self.kv = model.states.add_kv_layer(self.kv_heads, self.dim, self.vdim, _KV[model.act_dtype])
+            self.kv = model.states.add_kv_layer(self.kv_heads, self.dim, 0 if self.keys_as_values else self.vdim,
+                                                _KV[model.act_dtype], key_scale=self.keys_as_values)
         else:
             if getattr(self, "kv", None) is not None:
                 raise ValueError("a layer that borrows keys and values cannot run in a looped block")
             self.kv = self._src.kv
-        self.conv_state = model.states.add_state((self.taps - 1) * self.in_cols) if self.taps > 1 else None
+        self.conv_state = model.states.add_state((self.taps - 1) * self.qkv_cols) if self.taps > 1 else None
 
     def _prepare(self, c, proj, off):
         """Convolution and rotation of this step's q | k | v rows, then the new keys and values go to the pool.  Returns
@@ -484,12 +551,12 @@ class MaskedAttention:
         b, lib, s, R = c.batch, c.lib, _cabi.stream(), c.R
         if self.taps:
             chunks, nch, _s0, _sn = b.chunk_items(CONV_CHUNK)
-            y = c.empty(R, self.in_cols)
-            _chk(lib.pa_causal_conv(proj.data_ptr(), proj.stride(0), off, self.in_cols, self.taps, self.conv_w.data_ptr(),
-                                    None, 0, _cabi.ptr(self.conv_state), chunks.data_ptr(), nch, y.data_ptr(), self.in_cols,
+            y = c.empty(R, self.qkv_cols)
+            _chk(lib.pa_causal_conv(proj.data_ptr(), proj.stride(0), off, self.qkv_cols, self.taps, self.conv_w.data_ptr(),
+                                    None, 0, _cabi.ptr(self.conv_state), chunks.data_ptr(), nch, y.data_ptr(), self.qkv_cols,
                                     c.elem, s), "pa_causal_conv")
             if self.taps > 1:
-                _chk(lib.pa_conv_state_update(proj.data_ptr(), proj.stride(0), off, self.in_cols, self.taps,
+                _chk(lib.pa_conv_state_update(proj.data_ptr(), proj.stride(0), off, self.qkv_cols, self.taps,
                                               b.seq_start.data_ptr(), b.seq_len.data_ptr(), b.seq_slot.data_ptr(),
                                               b.num_seqs, self.conv_state.data_ptr(), c.elem, s), "pa_conv_state_update")
             proj, off = y, 0
@@ -505,6 +572,15 @@ class MaskedAttention:
                                        kv.value_buffer_.data_ptr() if own else None, pt.device_data().data_ptr(),
                                        pt.num_beams_, pt.num_tiles_, kv.total_pages_, kv.tile_size_, b.row_slot.data_ptr(),
                                        b.row_pos.data_ptr(), R, c.elem, s), "pa_rope_kv_append")
+        elif self.qk_norm:      # q in place, keys (and values) on their way into the pool: one launch
+            pt = kv.page_table_
+            _chk(lib.pa_qk_norm_kv_append(proj.data_ptr(), proj.stride(0), off, k_off, v_off, self.heads, self.kv_heads,
+                                          self.dim, self.vdim, self.q_gain.data_ptr(), self.k_gain.data_ptr(), c.model.eps,
+                                          kv.key_buffer_.data_ptr(),
+                                          None if self.keys_as_values else kv.value_buffer_.data_ptr(),
+                                          _cabi.ptr(kv.key_scale_), pt.device_data().data_ptr(), pt.num_beams_,
+                                          pt.num_tiles_, kv.total_pages_, kv.tile_size_, b.row_slot.data_ptr(),
+                                          b.row_pos.data_ptr(), R, c.elem, s), "pa_qk_norm_kv_append")
         elif self.own_kv:
             kv.append_rows(proj, k_off, v_off, b.row_slot, b.row_pos)
         return proj, off
@@ -512,32 +588,37 @@ class MaskedAttention:
     def attend(self, c, proj, off):
         """proj [R, stride] holds q | k | v of this step's rows from column `off`; appends k / v to the pool and
         returns the heads' outputs [R, heads * vdim]."""
+        gate = (proj, off + self.qkv_cols) if self.gate else (None, 0)
         proj, off = self._prepare(c, proj, off)
         out = c.empty(c.R, self.heads * self.vdim)
-        if not self._attend_tiles(c, proj, off, out, self.mma_tokens):
+        if not self._attend_tiles(c, proj, off, gate, out, self.mma_tokens):
             self.mma_tokens = 0     # a stride or an alignment the tensor-core kernel refuses: the float kernels
-            self._attend_tiles(c, proj, off, out, 0)
+            self._attend_tiles(c, proj, off, gate, out, 0)
         return out
 
-    def _attend_tiles(self, c, proj, off, out, mma_tokens):
+    def _attend_tiles(self, c, proj, off, gate, out, mma_tokens):
         b, lib, kv, s = c.batch, c.lib, self.kv, _cabi.stream()
         pt = kv.page_table_
         table = pt.device_data()
         out_rot = c.rope_table(self.vdim, self.rot_base) if self.rot_values else None
+        values = kv.key_buffer_ if self.keys_as_values else kv.value_buffer_
         for kind, group in b.query_tiles(self.tile_tokens, mma_tokens, MMA_FROM).items():
             if group is None:
                 continue
             tiles, ntiles, _longest = group
-            st = lib.pa_masked_attention_sink(proj.data_ptr(), proj.stride(0), off, kv.key_buffer_.data_ptr(),
-                                              kv.value_buffer_.data_ptr(), table.data_ptr(), pt.num_beams_, pt.num_heads_,
-                                              pt.num_tiles_, kv.total_pages_, kv.tile_size_, tiles.data_ptr(), ntiles,
-                                              self.heads, self.dim, self.vdim, self.scale, self.softcap, self.mask_kind,
-                                              self.mask_size, self.mask_keep, self.bias_kind, _cabi.ptr(self.bias),
-                                              self.bias_len, _cabi.ptr(self.head_scale), _cabi.ptr(self.sink),
-                                              _cabi.ptr(out_rot), out.data_ptr(), c.elem, kind, s)
+            st = lib.pa_masked_attention_gated(proj.data_ptr(), proj.stride(0), off, kv.key_buffer_.data_ptr(),
+                                               values.data_ptr(), table.data_ptr(), pt.num_beams_, pt.num_heads_,
+                                               pt.num_tiles_, kv.total_pages_, kv.tile_size_, tiles.data_ptr(), ntiles,
+                                               self.heads, self.dim, self.vdim, self.scale, self.softcap, self.mask_kind,
+                                               self.mask_size, self.mask_keep, self.bias_kind, _cabi.ptr(self.bias),
+                                               self.bias_len, _cabi.ptr(self.head_scale), _cabi.ptr(self.sink),
+                                               _cabi.ptr(out_rot), _cabi.ptr(kv.key_scale_), self.sigmoid,
+                                               _cabi.ptr(self.head_bias), _cabi.ptr(gate[0]),
+                                               gate[0].stride(0) if gate[0] is not None else 0, gate[1], out.data_ptr(),
+                                               c.elem, kind, s)
             if kind == 2 and st == _cabi.PA_ERR_UNSUPPORTED:
                 return False
-            _chk(st, "pa_masked_attention_sink")
+            _chk(st, "pa_masked_attention_gated")
         return True
 
     def project_out(self, c, heads_out):
@@ -545,44 +626,61 @@ class MaskedAttention:
 
 
 def decay_scan(c, state, out, heads, groups, dim, vdim, q, k, v, act=0, decay=None, dt=None, dt_bias=None, a_log=None,
-               skip=None):
+               skip=None, rope=None, rot_dims=0, k_scale=1.0):
     """The matrix-state recurrence of csrc/recurrence_ops.cu over this step's portions: q, k, v and dt are (buffer,
-    column offset) pairs; long portions take the chunked three-pass form."""
+    column offset) pairs; long portions take the chunked three-pass form.  rope: table of the rotation (halves) of the
+    first rot_dims dimensions of q and k; k_scale: a factor on k."""
     b, lib = c.batch, c.lib
     chunked = max(p[1] for p in b.portions) >= DECAY_CHUNKED_FROM
     items, n, s0, sn = b.chunk_items(DECAY_CHUNK if chunked else 0)
     ws = None
     if chunked:
         ws = c.empty(lib.pa_decay_scan_workspace_bytes(n, heads, dim, vdim), dtype=torch.uint8)
-    _chk(lib.pa_decay_scan(q[0].data_ptr(), q[0].stride(0), q[1], k[0].data_ptr(), k[0].stride(0), k[1], v[0].data_ptr(),
-                           v[0].stride(0), v[1], heads, groups, dim, vdim, act, _cabi.ptr(decay),
-                           dt[0].data_ptr() if dt else None, dt[0].stride(0) if dt else 0, dt[1] if dt else 0,
-                           _cabi.ptr(dt_bias), _cabi.ptr(a_log), _cabi.ptr(skip), state.data_ptr(), out.data_ptr(),
-                           out.stride(0), items.data_ptr(), n, s0.data_ptr(), sn.data_ptr(), b.seq_slot.data_ptr(),
-                           b.num_seqs, 1 if chunked else 0, _cabi.ptr(ws), ws.numel() if ws is not None else 0, c.elem,
-                           _cabi.stream()), "pa_decay_scan")
+    _chk(lib.pa_decay_scan_rotated(
+        q[0].data_ptr(), q[0].stride(0), q[1], k[0].data_ptr(), k[0].stride(0), k[1], v[0].data_ptr(), v[0].stride(0), v[1],
+        heads, groups, dim, vdim, act, _cabi.ptr(decay), dt[0].data_ptr() if dt else None, dt[0].stride(0) if dt else 0,
+        dt[1] if dt else 0, _cabi.ptr(dt_bias), _cabi.ptr(a_log), _cabi.ptr(skip), _cabi.ptr(rope), rot_dims, k_scale,
+        state.data_ptr(), out.data_ptr(), out.stride(0), items.data_ptr(), n, s0.data_ptr(), sn.data_ptr(),
+        b.seq_slot.data_ptr(), b.num_seqs, 1 if chunked else 0, _cabi.ptr(ws), ws.numel() if ws is not None else 0, c.elem,
+        _cabi.stream()), "pa_decay_scan_rotated")
 
 
 class DecayLinearAttention:
-    """Linear attention with a constant decay per head (cfg 'decay', one number per head): q, k, v = silu of their
-    projections, the matrix state per head and sequence in a float state slot, the heads' outputs normed together
-    (plain weight '<prefix>norm'), gated by sigmoid(W_g h), then the output product.  Reads q | k | v | g from a
-    projection buffer at a column offset."""
+    """Linear attention with a constant decay per head (cfg 'decay', one number per head): the matrix state per head and
+    sequence in a float state slot.  Reads q | k | v | g from a projection buffer at a column offset.  The design picks
 
-    def __init__(self, model, prefix, cfg, W):
+      act          'silu' on q, k and v, or None
+      rot          rotation (halves) of the first cfg rot.dims dimensions of q and k, in float inside the scan
+      key_scale    k times dim^(-1/2)
+      norm         'all': the heads' outputs normed together with the plain weight '<prefix>norm'; 'head': every head
+                   divided by its own root mean square, no weight
+      gate         'sigmoid' or 'silu' of W_g h on the normed outputs"""
+
+    def __init__(self, model, prefix, cfg, W, act="silu", rot=False, key_scale=False, norm="all", gate="sigmoid"):
         self.heads, self.dim, self.vdim = int(cfg["heads"]), int(cfg["dim"]), int(cfg["vdim"])
         H = self.heads
+        if act not in ("silu", None) or norm not in ("all", "head") or gate not in ("sigmoid", "silu"):
+            raise ValueError(f"{prefix}: unknown act {act!r}, norm {norm!r} or gate {gate!r}")
         if len(cfg["decay"]) != H:
             raise ValueError(f"{prefix}: one decay per head expected")
         shapes = (("q", H * self.dim), ("k", H * self.dim), ("v", H * self.vdim), ("g", H * self.vdim))
         for name, rows in shapes:
             if tuple(W[prefix + name].shape) != (rows, model.width):
                 raise ValueError(f"{prefix}{name}: shape does not match the config")
+        if tuple(W[prefix + "o"].shape) != (model.width, H * self.vdim):
+            raise ValueError(f"{prefix}o: shape does not match the config")
         self.in_weight = torch.cat([W[prefix + n] for n, _ in shapes], 0)
         self.in_bias = torch.zeros(self.in_weight.shape[0], dtype=self.in_weight.dtype, device=self.in_weight.device)
         self.in_cols = int(self.in_weight.shape[0])
         self.decay = model._f32(torch.tensor([float(d) for d in cfg["decay"]], dtype=torch.float64))
-        self.norm = model._f32(W[prefix + "norm"])
+        self.act = 1 if act == "silu" else 0
+        self.rot_dims, self.rot_base = (int(cfg["rot"]["dims"]), float(cfg["rot"]["base"])) if rot else (0, 0.0)
+        if self.rot_dims % 2 or self.rot_dims > self.dim:
+            raise ValueError(f"{prefix}: rot.dims must be even and at most dim")
+        self.k_scale = self.dim ** -0.5 if key_scale else 1.0
+        self.norm = model._f32(W[prefix + "norm"]) if norm == "all" else None
+        self.norm_groups = 1 if norm == "all" else H
+        self.gate_mode = 2 if gate == "sigmoid" else 3
         self.w_o = model._weight(W[prefix + "o"])
         self.alloc_state(model)
 
@@ -592,13 +690,32 @@ class DecayLinearAttention:
     def forward(self, c, proj, off):
         H, d, vd = self.heads, self.dim, self.vdim
         o = c.empty(c.R, H * vd, dtype=torch.float32)
-        decay_scan(c, self.state, o, H, H, d, vd, (proj, off), (proj, off + H * d), (proj, off + 2 * H * d), act=1,
-                   decay=self.decay)
+        decay_scan(c, self.state, o, H, H, d, vd, (proj, off), (proj, off + H * d), (proj, off + 2 * H * d), act=self.act,
+                   decay=self.decay, rope=c.rope_table(self.rot_dims, self.rot_base), rot_dims=self.rot_dims,
+                   k_scale=self.k_scale)
         on = c.empty(c.R, H * vd)
-        _chk(c.lib.pa_gated_rms_norm(o.data_ptr(), c.R, H * vd, 1, proj.data_ptr(), proj.stride(0), off + 2 * H * d + H * vd, 2,
-                                     self.norm.data_ptr(), c.model.eps, on.data_ptr(), c.elem, _cabi.stream()),
-             "pa_gated_rms_norm")
+        _chk(c.lib.pa_gated_rms_norm(o.data_ptr(), c.R, H * vd, self.norm_groups, proj.data_ptr(), proj.stride(0),
+                                     off + 2 * H * d + H * vd, self.gate_mode, _cabi.ptr(self.norm), c.model.eps, on.data_ptr(),
+                                     c.elem, _cabi.stream()), "pa_gated_rms_norm")
         return c.model._linear(on, self.w_o)
+
+
+class LinearAttentionMixer:
+    """A DecayLinearAttention as a layer's only mixer: one fused q | k | v | g product, scan, norm and gate, output product."""
+    kind = "retention"
+
+    def __init__(self, model, prefix, cfg, W, **constants):
+        self.core = DecayLinearAttention(model, prefix, cfg, W, **constants)
+        self.w_in = model._weight(self.core.in_weight)
+
+    def new_pass(self, model):
+        m = copy.copy(self)
+        m.core = copy.copy(self.core)
+        m.core.alloc_state(model)
+        return m
+
+    def forward(self, c, h):
+        return self.core.forward(c, c.model._linear(h, self.w_in), 0)
 
 
 class SoftmaxAttentionMixer:
@@ -851,7 +968,7 @@ DESIGNS = {
                                             "moe": dict(score="sigmoid", weight_on="input", act="silu", gated=True)}),
     "Domilix": dict(wiring="post_norm", ff={"dense": dict(act="relu", gated=True),
                                             "moe": dict(score="softmax_chosen", weight_on="output", act="relu2", gated=False)}),
-    "Dubarax": dict(wiring="pre_norm",
+    "Dubarax": dict(wiring="pre_norm", loop_entry=True,
                     mixers={"attention": (SoftmaxAttentionMixer, dict(mask="window", bias="bucket", softcap=True)),
                             "parallel": (ParallelMixer, dict(left=dict(mask="chunk", bias="slope", slope_exp=8.0))),
                             "mamba2": (Mamba2Mixer, {})},
@@ -864,6 +981,12 @@ DESIGNS = {
                      ff={"dense": dict(act="poly_norm", gated=False, bias=True),
                          "moe": dict(score="softmax", weight_on="output", act="silu", gated=True, correction=True,
                                      renorm=True)}),
+    "Namudra": dict(wiring="streams",
+                    mixers={"retention": (LinearAttentionMixer, dict(act=None, rot=True, key_scale=True, norm="head", gate="silu")),
+                            "attention": (SoftmaxAttentionMixer, dict(mask="window", proj_bias=False, qk_norm=True, values="keys",
+                                                                      weights="sigmoid", head_bias=True, gate=True)),
+                            "latent_attention": (LatentAttentionMixer, dict(pairing="halves", head_gate=False))},
+                    ff={"dense": dict(act="silu", gated=True)}),
 }
 
 
@@ -894,7 +1017,10 @@ class HybridDecoder:
             raise ValueError("embed does not match config vocab / width")
         self.embed = W["embed"].to(self.device, self.act_dtype).contiguous()
         self.head = self._weight(W["head"])
-        post, pre, par2 = self.wiring == "post_norm", self.wiring == "pre_norm", self.wiring == "parallel_two_norms"
+        self.streams = int(config.get("streams") or 0)
+        if self.wiring == "streams" and self.streams == 0:
+            self.wiring = "pre_norm"        # a single residual without stream mixing
+        post, pre, par2 = self.wiring == "post_norm", self.wiring in ("pre_norm", "streams"), self.wiring == "parallel_two_norms"
         self.final_gain = 1.0 if post or pre or par2 else float(W["final.norm"].to(torch.float32))
         self.final_gain_vec = (self._f32(W["final.norm"].reshape(-1)) if post or par2 else
                                self._gain1p(W["final.norm"]) if pre else None)
@@ -915,6 +1041,9 @@ class HybridDecoder:
                 L.gain1 = self._gain1p(W[p + "norm1"])
                 L.gain2 = self._gain1p(W[p + "norm2"]) if lc.get("mlp") else None
                 L.shift = L.prev = None
+                if self.wiring == "streams":
+                    L.hc1 = self._stream_weights(W, p + "hc1.")
+                    L.hc2 = self._stream_weights(W, p + "hc2.") if lc.get("mlp") else None
             else:
                 L.gain = float(W[p + "norm1"].to(torch.float32))
                 L.shift = self._f32(W[p + "shift"]) if p + "shift" in W else None
@@ -937,28 +1066,31 @@ class HybridDecoder:
     def _build_runs(self, loop, W):
         """The order in which layers RUN: (layer, mixer, pass number or None).  A looped block [start, stop) runs `times`
         times in a row with the same weights; every pass after the first gets mixers with a cache / state of their own
-        (new_pass), and its first run carries the pass number: the block input x <- W_in [x | x0] + step[t] comes first."""
+        (new_pass).  In a design with `loop_entry` its first run carries the pass number: the block input
+        x <- W_in [x | x0] + step[t] comes first."""
         n = len(self.layers)
         self.loop_in = self.loop_step = None
         if not loop or int(loop.get("times", 0)) < 1 or int(loop["stop"]) <= int(loop["start"]):
             self.runs = [(L, L.mixer, None) for L in self.layers]
             return
-        if self.wiring != "pre_norm":
-            raise ValueError("looped blocks are served in the pre-norm wiring")
+        if self.wiring not in ("pre_norm", "streams"):
+            raise ValueError("looped blocks are served in the pre-norm and stream wirings")
         a, b, times = int(loop["start"]), int(loop["stop"]), int(loop["times"])
         if not 0 <= a < b <= n:
             raise ValueError("loop: start / stop outside the layer list")
-        if tuple(W["loop.in"].shape) != (self.width, 2 * self.width) or tuple(W["loop.step"].shape) != (times, self.width):
-            raise ValueError("loop.in / loop.step do not match width / times")
-        self.loop_in = self._weight(W["loop.in"])
-        self.loop_step = self._f32(W["loop.step"])
+        entry = bool(self.design.get("loop_entry"))
+        if entry:
+            if tuple(W["loop.in"].shape) != (self.width, 2 * self.width) or tuple(W["loop.step"].shape) != (times, self.width):
+                raise ValueError("loop.in / loop.step do not match width / times")
+            self.loop_in = self._weight(W["loop.in"])
+            self.loop_step = self._f32(W["loop.step"])
         self.runs = [(L, L.mixer, None) for L in self.layers[:a]]
         for t in range(times):
             for i in range(a, b):
                 L = self.layers[i]
                 if t and not hasattr(L.mixer, "new_pass"):
                     raise ValueError(f"mixer {L.mixer.kind!r} cannot run in a looped block")
-                self.runs.append((L, L.mixer if t == 0 else L.mixer.new_pass(self), t if i == a else None))
+                self.runs.append((L, L.mixer if t == 0 else L.mixer.new_pass(self), t if entry and i == a else None))
         self.runs += [(L, L.mixer, None) for L in self.layers[b:]]
 
     @classmethod
@@ -974,6 +1106,13 @@ class HybridDecoder:
     def _gain1p(self, t):
         """1 + w of a norm weight stored around zero (float)."""
         return (1.0 + t.reshape(-1).to(torch.float32)).to(self.device).contiguous()
+
+    def _stream_weights(self, W, p):
+        """Weights of a sublayer over residual streams: (in [s], out [s], mix [from][to]) in float."""
+        S = self.streams
+        if tuple(W[p + "in"].shape) != (S,) or tuple(W[p + "out"].shape) != (S,) or tuple(W[p + "mix"].shape) != (S, S):
+            raise ValueError(f"{p}in / out / mix do not match the number of streams")
+        return tuple(self._f32(W[p + n]) for n in ("in", "out", "mix"))
 
     def _bias(self, t):
         """A linear layer's bias for _linear: the activation type for the vendor GEMM's epilogue, float for the fp32 kernel."""
@@ -1024,6 +1163,8 @@ class HybridDecoder:
             x = self._pre_norm_layers(c, x)
         elif self.wiring == "parallel_two_norms":
             self._parallel_two_norm_layers(c, x)
+        elif self.wiring == "streams":
+            return self._logits(self._stream_layers(c, x, want_rows))
         for L in self.layers if self.wiring == "parallel" else ():
             h = c.empty(R, W)
             hs = c.empty(R, W) if L.shift is not None else None
@@ -1052,10 +1193,16 @@ class HybridDecoder:
         hf = torch.empty((n, W), dtype=self.act_dtype, device=self.device)
         _chk(lib.pa_rms_norm_shift(xs.data_ptr(), n, W, self.eps, self.final_gain, _cabi.ptr(self.final_gain_vec), None, None,
                                    None, None, hf.data_ptr(), None, c.elem, s), "pa_rms_norm_shift")
+        return self._logits(hf)
+
+    def _logits(self, hf):
+        """Float logits of final-normed rows (activation type)."""
+        if hf.shape[0] == 0:
+            return torch.empty((0, self.vocab), dtype=torch.float32, device=self.device)
         logits = self._linear(hf, self.head, out_dtype=torch.float32)
         if self.logit_scale != 1.0 or self.logit_softcap > 0.0:
-            _chk(lib.pa_logit_softcap(logits.data_ptr(), logits.numel(), self.logit_scale, self.logit_softcap, s),
-                 "pa_logit_softcap")
+            _chk(self._lib.pa_logit_softcap(logits.data_ptr(), logits.numel(), self.logit_scale, self.logit_softcap,
+                                            _cabi.stream()), "pa_logit_softcap")
         return logits
 
     def _parallel_two_norm_layers(self, c, x):
@@ -1156,4 +1303,42 @@ class HybridDecoder:
         add_norm(x, pending, None)
         return x
 
-    layer_hook = None   # debugging aid: called with the float residual after every layer
+    def _stream_layers(self, c, x, want_rows):
+        """The residual as `streams` float rows per token, all equal to the embedding at the start.  Per sublayer:
+        u = sum_s in[s] x_s;  y = f(N(u));  x_t <- sum_s mix[s][t] x_s + out[t] y.  pa_streams_add_norm applies one sublayer's
+        update and leaves the NEXT sublayer's operand in the same pass; before the first update it reads the embedding
+        row for every stream, and after the last it keeps no streams: the final norm of the sum of the wanted rows' streams
+        comes out directly.  Returns the final-normed rows in the activation type."""
+        lib, R, W, S, s = self._lib, c.R, self.width, self.streams, _cabi.stream()
+        cur = dict(x=x, n=1)            # the current streams: [R][n][W]
+
+        def advance(y, hc, in_w=None, gain=None, keep=True, rows=None, want_sum=False):
+            n = rows.numel() if rows is not None else R
+            dst = None
+            if y is not None and keep:
+                dst = cur["x"] if cur["n"] == S else torch.empty((R, S, W), dtype=torch.float32, device=self.device)
+            h = c.empty(n, W) if gain is not None else None
+            u = torch.empty((n, W), dtype=torch.float32, device=self.device) if want_sum else None
+            _chk(lib.pa_streams_add_norm(cur["x"].data_ptr(), cur["n"], _cabi.ptr(dst), n, S, W, _cabi.ptr(y),
+                                         _cabi.ptr(hc[2]) if hc else None, _cabi.ptr(hc[1]) if hc else None, _cabi.ptr(in_w),
+                                         self.eps, _cabi.ptr(gain), _cabi.ptr(u), _cabi.ptr(h), _cabi.ptr(rows), c.elem, s),
+                 "pa_streams_add_norm")
+            if dst is not None:
+                cur.update(x=dst, n=S)
+            return u if want_sum else h
+
+        y = hc = None                   # the output of the last sublayer that is not in the streams yet, and its weights
+        for L, mixer, _pass in self.runs:
+            y, hc = mixer.forward(c, advance(y, hc, L.hc1[0], L.gain1)), L.hc1
+            if L.ff is not None:
+                ff = L.ff.forward(c, advance(y, hc, L.hc2[0], L.gain2))
+                y, hc = ff["dense"], L.hc2
+            if self.layer_hook is not None:
+                total = advance(y, hc, want_sum=True)
+                y = hc = None
+                self.layer_hook(total)
+        if want_rows is not None and want_rows.numel() == 0:
+            return c.empty(0, W)
+        return advance(y, hc, gain=self.final_gain_vec, keep=False, rows=want_rows)
+
+    layer_hook = None   # debugging aid: called with the float residual (the sum of its streams) after every layer

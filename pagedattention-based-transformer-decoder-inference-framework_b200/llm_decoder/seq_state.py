@@ -113,13 +113,16 @@ class SequenceStateCache:
         self._states.append(t)
         return t
 
-    def add_kv_layer(self, kv_heads, key_dim, value_dim, dtype):
+    def add_kv_layer(self, kv_heads, key_dim, value_dim, dtype, key_scale=False):
         """A paged pool for one attention layer: max_tiles * kv_heads pages; the table has one row per slot and lets a
-        single request grow to the whole pool."""
+        single request grow to the whole pool.  key_scale: a float per key beside the pool (key_scale_, by pool row)."""
         kvc = KVTileCache(dtype, device=self.device)
         kvc.init(self.max_tiles * int(kv_heads), self.tile_size, int(key_dim), int(value_dim))
         kvc.configure_table(self.max_seqs, int(kv_heads), self.max_tiles)
         kvc.evict_on_exhaustion = False
+        kvc.key_scale_ = None
+        if key_scale:
+            kvc.key_scale_ = torch.zeros(kvc.total_pages_ * self.tile_size, dtype=torch.float32, device=self.device)
         self._kv.append(kvc)
         return kvc
 
