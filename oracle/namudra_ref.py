@@ -266,7 +266,10 @@ def random_weights(config, seed=0):
             W[m + "uk"], W[m + "uv"], W[m + "o"] = mat(H * d, kr), mat(H * e, kr), mat(Wd, H * e)
         else:
             d, e = c["dim"], c["vdim"]
-            W[m + "q"], W[m + "k"], W[m + "v"] = mat(H * d, Wd), mat(H * d, Wd), mat(H * e, Wd)
+            W[m + "q"], W[m + "v"] = mat(H * d, Wd), mat(H * e, Wd)
+            # keys that lean towards the queries: a token meets its own key with a score well above zero, so the norm of a
+            # head (no weight, small eps) does not blow up the rounding of a nearly empty state
+            W[m + "k"] = (0.8 * W[m + "q"].float() + mat(H * d, Wd, 0.6).float()).to(torch.bfloat16)
             W[m + "g"], W[m + "o"] = mat(H * e, Wd), mat(Wd, H * e)
         if lc.get("mlp"):
             ff = lc["mlp"]["ff"]
