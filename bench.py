@@ -31,6 +31,8 @@ extra  = the other BASELINE.json configurations under the same clock (benchmarks
          windowed / chunked attention, linear attention, a state-space mixer, group-limited experts) next to `Megusun`.
 --gunulorn: likewise (benchmarks/gunulorn.py): the stack serving the `Gunulorn` design (two-norm parallel wiring, attention
          with convolved projections / sinks / a kept prefix / turned values, PolyNorm, identity experts) next to `Dubarax`.
+--namudra: likewise (benchmarks/namudra.py): the stack serving the `Namudra` design (residual streams, windowed sigmoid
+         attention whose values are its keys, latent attention, rotated retention) next to `Dubarax` and `Domilix`.
 N > 1: one process per GPU (torchrun), rows sharded across ranks, no data-path collective in the headline
          step; c5_splitkv is the mode with an exchange.
 """
@@ -81,6 +83,11 @@ def parse():
                          "the Gunulorn design at realistic layer sizes next to the Dubarax design at equal size, and its "
                          "kernels next to the like kernels of that design against their rooflines (benchmarks/gunulorn.py); "
                          "one JSON line")
+    ap.add_argument("--namudra", action="store_true",
+                    help="instead of the headline workload: prefill / decode throughput of the config-driven stack serving "
+                         "the Namudra design at realistic layer sizes next to the Dubarax and Domilix designs at equal size, "
+                         "and its kernels next to the like kernels of those designs against their rooflines "
+                         "(benchmarks/namudra.py); one JSON line")
     ap.add_argument("--latent", action="store_true",
                     help="instead of the headline workload: prefill / decode throughput of the config-driven stack serving "
                          "the Domilix design (latent attention) at realistic layer sizes next to the Megusun design at "
@@ -470,6 +477,10 @@ def main():
     if args.gunulorn:
         from benchmarks import gunulorn
         print(json.dumps({"bench": "gunulorn", **gunulorn.run()}, default=float))
+        return
+    if args.namudra:
+        from benchmarks import namudra
+        print(json.dumps({"bench": "namudra", **namudra.run()}, default=float))
         return
     if args.latent:
         from benchmarks import latent
