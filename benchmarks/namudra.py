@@ -200,7 +200,7 @@ def bench_kernels(s, dev, only=None):
                 continue
             tiles, ntiles, _longest = group
 
-            def attend(x, pool, vals, cap, bias, ks, sig, hb, gate_off):
+            def attend(x, pool, vals, cap, bias, ks, sig, hb, gate_off, kind=3 if kind == 1 else kind):
                 pt = pool.page_table_
                 return lib.pa_masked_attention_gated(
                     x.data_ptr(), x.stride(0), 0, pool.key_buffer_.data_ptr(), vals.data_ptr(), pt.device_data().data_ptr(), pt.num_beams_,
@@ -218,6 +218,10 @@ def bench_kernels(s, dev, only=None):
                 rec(f"window_sigmoid_keys_as_values/{tag}", mine, bytes_=nseq * seen * G * (D * 2 + 4))
                 rec(f"window_bucket_cap~/{tag}", other, bytes_=nseq * seen * G * D * 4)
                 rec(f"window_plain_softmax~/{tag}", plain, bytes_=nseq * seen * G * D * 4)
+                rec(f"window_sigmoid_keys_as_values streaming/{tag}", lambda: attend(
+                    proj, kv, kv.key_buffer_, 0.0, None, kv.key_scale_, 1, pb, H * D + G * D, 1), bytes_=nseq * seen * G * (D * 2 + 4))
+                rec(f"window_bucket_cap~ streaming/{tag}", lambda: attend(
+                    qkv, kv2, kv2.value_buffer_, 30.0, bucket, None, 0, None, None, 1), bytes_=nseq * seen * G * D * 4)
         gq, gk = torch.ones(D, device=dev), torch.ones(D, device=dev)
         pt, pt2, ptl = kv.page_table_, kv2.page_table_, kvl.page_table_
         rec(f"qk_norm_kv_append/{tag}", lambda: lib.pa_qk_norm_kv_append(

@@ -815,7 +815,9 @@ int pa_gated_rms_norm(const float* d_y, int64_t rows, int inner, int groups, con
  *   per pool row on the dot product; sigmoid_weights 1: the weight of a visible key is sigmoid(score) and nothing divides
  *   the sum (no sink then); d_head_bias [heads] (NULL: none) added to the score last; d_gate (NULL: none): rows of the
  *   activation type, output column c of head h is multiplied by sigmoid(gate[row * gate_stride + gate_off + h * vdim + c])
- *   in float before it is rounded.  d_v_pool == d_k_pool (dim == vdim): the values are the cached key rows, read once.
+ *   in float before it is rounded.  tile_kind 3: every tile is ONE token (decoded tokens) and the query heads of a kv head
+ *   are the rows of tensor-core products (bfloat16, the shapes of tile_kind 2; PA_ERR_UNSUPPORTED otherwise); meant for
+ *   batches with at least one (token, kv head) pair per SM.  d_v_pool == d_k_pool (dim == vdim): the values are the cached key rows, read once.
  * pa_qk_norm_kv_append: query head h (columns q_off + h * dim) is divided by its root mean square and multiplied by
  *   d_q_gain [dim], in place; the key of kv head g (k_off + g * dim) goes to the row's place in the pool: normed likewise
  *   (d_k_gain) where d_key_scale is NULL, else as it is, with its inverse root mean square in d_key_scale (the key norm's

@@ -165,7 +165,6 @@ struct MaskAttnParams {
     const float* sink;          // [heads] or null
     int mask_keep;              // window masks: the first mask_keep positions stay visible
     const float* out_rot;       // [rows][vdim / 2][2] or null
-    int head_rows;              // tensor-core kernel: every tile is ONE token and the rows are the heads of a kv head
     int sigm;                   // 1: weight = sigmoid(score), nothing divides the sum (no sink)
     const float* key_scale;     // [total_pages * tile_size] or null
     const float* head_bias;     // [heads] or null
@@ -724,7 +723,7 @@ __global__ void __launch_bounds__(kMmThreads) masked_attention_mma_kernel(const 
         const int64_t pr = pool_row(kt * kMmKeys + key);
         if (q2 == 0) {
             key_ok[buf][key] = pr >= 0;
-            if (p.key_scale) key_sc[buf][key] = pr >= 0 ? p.key_scale[pr] : 0.f;
+            if (p.key_scale) cp_async_4(smem_u32(&key_sc[buf][key]), p.key_scale + (pr >= 0 ? pr : 0), pr >= 0);
         }
         bf16_t* kdst = Ks + (buf * kMmKeys + key) * KS;
         const bf16_t* ksrc = kp + (pr >= 0 ? pr * dim : 0);
@@ -921,10 +920,14 @@ static int mm_launch(const MaskAttnParams& p, int ntiles, cudaStream_t st) {
 static bool mm_shape_ok(int dim, int vdim) { return dim % 8 == 0 && dim <= 128 && vdim % 8 == 0 && vdim <= 128; }
 static int mm_padded(int n) { return n <= 32 ? 32 : n <= 64 ? 64 : 128; }
 
+static bool mm_operands_ok(const MaskAttnParams& p) {
+    return mm_shape_ok(p.dim, p.vdim) && p.q_stride % 8 == 0 && p.q_off % 8 == 0 && (uintptr_t)p.q % 16 == 0 &&
+           (uintptr_t)p.k_pool % 16 == 0 && (uintptr_t)p.v_pool % 16 == 0 && (uintptr_t)p.out % 4 == 0;
+}
+
 // PA_ERR_UNSUPPORTED: this shape or these pointers stay on the float kernel
 static int mm_dispatch(const MaskAttnParams& p, int ntiles, cudaStream_t st) {
-    if (!mm_shape_ok(p.dim, p.vdim) || p.q_stride % 8 || p.q_off % 8) return PA_ERR_UNSUPPORTED;
-    if ((uintptr_t)p.q % 16 || (uintptr_t)p.k_pool % 16 || (uintptr_t)p.v_pool % 16 || (uintptr_t)p.out % 4) return PA_ERR_UNSUPPORTED;
+    if (!mm_operands_ok(p)) return PA_ERR_UNSUPPORTED;
     const int dp = mm_padded(p.dim), vp = mm_padded(p.vdim);
     if (p.k_pool == p.v_pool) {
 #define PA_MM_CASE(D) if (dp == D) return p.sigm ? mm_launch<D, D, true, true>(p, ntiles, st) : mm_launch<D, D, false, true>(p, ntiles, st)
@@ -937,6 +940,268 @@ static int mm_dispatch(const MaskAttnParams& p, int ntiles, cudaStream_t st) {
     PA_MM_CASE(64, 32); PA_MM_CASE(64, 64); PA_MM_CASE(64, 128);
     PA_MM_CASE(128, 32); PA_MM_CASE(128, 64); PA_MM_CASE(128, 128);
 #undef PA_MM_CASE
+    return PA_ERR_UNSUPPORTED;
+}
+
+// ---- decoded tokens on the tensor cores (bfloat16) ---------------------------------------------------------------------
+// One CTA = one token x one key/value head x up to 16 of its query heads, which are the ROWS of the products.  The staged
+// tiles are those of the portion kernel (64 keys, 16-byte cp.async copies, a ring of three or five buffers); the four warps split the 64
+// keys of a step, 16 each, keep a running (m, l, o) of their own and meet in shared memory at the end.  Every cached row is
+// read once, in whole lines, whatever the number of heads; for batches with at least one CTA per SM.
+constexpr int kMdRows = 16;
+constexpr int md_stages(bool shared) { return shared ? 5 : 3; }     // two resident CTAs per SM at 128-wide heads
+
+template <int DIM, int VDIM, bool SHARED>
+__global__ void __launch_bounds__(kMmThreads) masked_attention_mma_decode_kernel(const MaskAttnParams p) {
+    static_assert(!SHARED || DIM == VDIM, "values that are the keys have their size");
+    constexpr int KS = DIM + kMmPad, VS = VDIM + kMmPad, NT = VDIM / 8, NST = md_stages(SHARED), OS = VDIM + 4;
+    extern __shared__ __align__(16) unsigned char mm_smem[];
+    bf16_t* Qs = reinterpret_cast<bf16_t*>(mm_smem);         // [16][KS]
+    bf16_t* Ks = Qs + kMdRows * KS;                           // [NST][64][KS]
+    bf16_t* Vs = SHARED ? Ks : Ks + NST * kMmKeys * KS;       // [NST][64][VS]
+    float* Os = reinterpret_cast<float*>(Ks);                 // [4][16][OS], over the tiles once they are consumed
+    __shared__ int key_ok[NST][kMmKeys];
+    __shared__ __align__(8) float key_sc[NST][kMmKeys];
+    __shared__ float ms[4][kMdRows], ls[4][kMdRows];
+
+    const int hpg = p.heads / p.num_kv_heads, nchunk = (hpg + kMdRows - 1) / kMdRows;
+    const int* tile = p.tiles + 4 * blockIdx.x;
+    const int row0 = tile[0], slot = tile[2], pos = tile[3];
+    const int g = blockIdx.y / nchunk, hbase = g * hpg + blockIdx.y % nchunk * kMdRows;
+    const int nrow = min(kMdRows, (g + 1) * hpg - hbase);     // query heads of this CTA
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const bf16_t* kp = static_cast<const bf16_t*>(p.k_pool);
+    const bf16_t* vp = static_cast<const bf16_t*>(p.v_pool);
+    const int32_t* trow = p.table + ((int64_t)slot * p.num_kv_heads + g) * p.num_tiles;
+    const int total = pos + 1, dim = p.dim, vdim = p.vdim;
+    const MaSteps steps = ma_steps(p, ma_first_key(p, pos), total, kMmKeys);
+
+    for (int c = tid; c < kMdRows * (DIM / 8); c += kMmThreads) {
+        const int r = c / (DIM / 8), cv = (c % (DIM / 8)) * 8;
+        const bool ok = r < nrow && cv < dim;
+        const bf16_t* src = static_cast<const bf16_t*>(p.q) + (ok ? (int64_t)row0 * p.q_stride + p.q_off + (int64_t)(hbase + r) * dim + cv : 0);
+        cp_async_16(smem_u32(Qs + r * KS + cv), src, ok);
+    }
+    // two threads per key; the page of a step's key is looked up one step before its copies are issued
+    const int key = tid >> 1, q2 = tid & 1;
+    auto look_up = [&](int sn) -> int64_t {
+        if (sn >= steps.count) return -1;
+        const int j = steps.step(sn) * kMmKeys + key;
+        if (j < total && ma_visible(p, pos, j) && j / p.tile_size < p.num_tiles) {
+            const int page = trow[j / p.tile_size];
+            if (page >= 0 && page < p.total_pages) return (int64_t)page * p.tile_size + j % p.tile_size;
+        }
+        return -1;
+    };
+    auto load_tile = [&](int64_t pr, int buf) {
+        if (q2 == 0) {
+            key_ok[buf][key] = pr >= 0;
+            if (p.key_scale) cp_async_4(smem_u32(&key_sc[buf][key]), p.key_scale + (pr >= 0 ? pr : 0), pr >= 0);
+        }
+        bf16_t* kdst = Ks + (buf * kMmKeys + key) * KS;
+        const bf16_t* ksrc = kp + (pr >= 0 ? pr * dim : 0);
+#pragma unroll
+        for (int i = 0; i < DIM / 16; ++i) {
+            const int cv = (q2 + 2 * i) * 8;
+            const bool ok = pr >= 0 && cv < dim;
+            cp_async_16(smem_u32(kdst + cv), ok ? ksrc + cv : kp, ok);
+        }
+        if (SHARED) return;
+        bf16_t* vdst = Vs + (buf * kMmKeys + key) * VS;
+        const bf16_t* vsrc = vp + (pr >= 0 ? pr * vdim : 0);
+#pragma unroll
+        for (int i = 0; i < VDIM / 16; ++i) {
+            const int cv = (q2 + 2 * i) * 8;
+            const bool ok = pr >= 0 && cv < vdim;
+            cp_async_16(smem_u32(vdst + cv), ok ? vsrc + cv : vp, ok);
+        }
+    };
+#pragma unroll
+    for (int t = 0; t < NST - 1; ++t) {
+        if (t < steps.count) load_tile(look_up(t), t);
+        cp_async_commit();
+    }
+    int64_t ahead = look_up(NST - 1);
+
+    float o[NT][4], m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+#pragma unroll
+    for (int t = 0; t < NT; ++t)
+#pragma unroll
+        for (int c = 0; c < 4; ++c) o[t][c] = 0.f;
+    const int r0 = lane >> 2;                                 // this thread's rows: r0 and r0 + 8
+    const float inv_cap = p.softcap > 0.f ? 1.0f / p.softcap : 0.f;
+    float slope[2], hfac[2], hbias[2];                        // of the two rows' heads
+    const float* btab[2];
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+        const int h = hbase + min(r0 + 8 * i, nrow - 1);
+        slope[i] = p.bias_kind == 1 ? p.bias[h] : 0.f;
+        hfac[i] = p.scale * (p.head_scale ? p.head_scale[h] : 1.f);
+        hbias[i] = p.head_bias ? p.head_bias[h] : 0.f;
+        btab[i] = p.bias_kind == 2 ? p.bias + h : nullptr;
+    }
+
+    for (int sn = 0; sn < steps.count; ++sn) {
+        const int buf = sn % NST, c0 = steps.step(sn) * kMmKeys;
+        if (sn + NST - 1 < steps.count) load_tile(ahead, (sn + NST - 1) % NST);
+        cp_async_commit();
+        ahead = look_up(sn + NST);
+        cp_async_wait<NST - 1>();
+        __syncthreads();
+        float s[2][4];
+#pragma unroll
+        for (int t = 0; t < 2; ++t)
+#pragma unroll
+            for (int c = 0; c < 4; ++c) s[t][c] = 0.f;
+        const bf16_t* kw = Ks + (buf * kMmKeys + warp * 16) * KS;
+#pragma unroll
+        for (int ks = 0; ks < DIM; ks += 16) {
+            if (ks >= dim) continue;                         // all padding
+            uint32_t a[4], b0, b1, b2, b3;
+            ldsm_x4(smem_u32(Qs + (lane & 15) * KS + ks + (lane >> 4) * 8), a[0], a[1], a[2], a[3]);
+            ldsm_x4(smem_u32(kw + ((lane & 7) + ((lane >> 4) << 3)) * KS + ks + ((lane >> 3) & 1) * 8), b0, b1, b2, b3);
+            mma_bf16_16816(s[0], a, b0, b1);
+            mma_bf16_16816(s[1], a, b2, b3);
+        }
+        float mx[2] = {-INFINITY, -INFINITY};
+#pragma unroll
+        for (int t = 0; t < 2; ++t) {
+            const int col = warp * 16 + t * 8 + 2 * (lane & 3);
+            const int2 okk = *reinterpret_cast<const int2*>(&key_ok[buf][col]);
+            const float2 ksc = p.key_scale ? *reinterpret_cast<const float2*>(&key_sc[buf][col]) : make_float2(1.f, 1.f);
+#pragma unroll
+            for (int c = 0; c < 4; ++c) {
+                const int i = c >> 1, dist = pos - (c0 + col + (c & 1));
+                const bool vis = ((c & 1) ? okk.y : okk.x) && r0 + 8 * i < nrow;
+                float v = s[t][c] * ((c & 1) ? ksc.y : ksc.x) * hfac[i];
+                if (p.softcap > 0.f) v = p.softcap * ma_tanh(v * inv_cap);
+                if (p.bias_kind == 1) v -= slope[i] * (float)dist;
+                else if (p.bias_kind == 2) v += btab[i][(int64_t)min(max(dist, 0), p.bias_len - 1) * p.heads];
+                s[t][c] = vis ? v + hbias[i] : -INFINITY;
+                mx[i] = fmaxf(mx[i], s[t][c]);
+            }
+        }
+        if (p.sigm) {
+#pragma unroll
+            for (int t = 0; t < 2; ++t)
+#pragma unroll
+                for (int c = 0; c < 4; ++c) s[t][c] = s[t][c] == -INFINITY ? 0.f : __fdividef(1.0f, 1.0f + __expf(-s[t][c]));
+        } else {
+#pragma unroll
+            for (int i = 0; i < 2; ++i) {
+                mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], 1));
+                mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], 2));
+                const float mn = fmaxf(m[i], mx[i]), ref = mn == -INFINITY ? 0.f : mn;
+                const float corr = __expf(m[i] - ref);       // m = -inf: 0 (nothing accumulated yet)
+                m[i] = mn;
+                l[i] *= corr;
+#pragma unroll
+                for (int t = 0; t < NT; ++t) {
+                    o[t][2 * i] *= corr;
+                    o[t][2 * i + 1] *= corr;
+                }
+#pragma unroll
+                for (int t = 0; t < 2; ++t)
+#pragma unroll
+                    for (int c = 2 * i; c < 2 * i + 2; ++c) {
+                        s[t][c] = __expf(s[t][c] - ref);
+                        l[i] += s[t][c];
+                    }
+            }
+        }
+        uint32_t a[4] = {pack_bf16x2(s[0][0], s[0][1]), pack_bf16x2(s[0][2], s[0][3]), pack_bf16x2(s[1][0], s[1][1]), pack_bf16x2(s[1][2], s[1][3])};
+        const bf16_t* vw = Vs + (buf * kMmKeys + warp * 16) * VS;
+#pragma unroll
+        for (int np = 0; np < NT / 2; ++np) {
+            if (np * 16 >= vdim) continue;                   // all padding
+            uint32_t b0, b1, b2, b3;
+            ldsm_x4_trans(smem_u32(vw + ((lane & 7) + ((lane >> 3) & 1) * 8) * VS + np * 16 + (lane >> 4) * 8), b0, b1, b2, b3);
+            mma_bf16_16816(o[2 * np], a, b0, b1);
+            mma_bf16_16816(o[2 * np + 1], a, b2, b3);
+        }
+        __syncthreads();                                     // this buffer is free for the copies of step sn + NST
+    }
+    cp_async_wait<0>();
+    __syncthreads();
+    // ---- the warps' partial results -> shared memory
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+        l[i] += __shfl_xor_sync(0xffffffffu, l[i], 1);
+        l[i] += __shfl_xor_sync(0xffffffffu, l[i], 2);
+        if ((lane & 3) == 0) { ms[warp][r0 + 8 * i] = m[i]; ls[warp][r0 + 8 * i] = l[i]; }
+        float* dst = Os + (warp * kMdRows + r0 + 8 * i) * OS + 2 * (lane & 3);
+#pragma unroll
+        for (int t = 0; t < NT; ++t) *reinterpret_cast<float2*>(dst + t * 8) = make_float2(o[t][2 * i], o[t][2 * i + 1]);
+    }
+    __syncthreads();
+    for (int idx = tid; idx < nrow * (vdim >> 1); idx += kMmThreads) {
+        const int r = idx / (vdim >> 1), col = idx % (vdim >> 1) * 2;
+        float f[4], inv = 1.f;
+        if (p.sigm) {
+            f[0] = f[1] = f[2] = f[3] = 1.f;
+        } else {
+            float M = fmaxf(fmaxf(ms[0][r], ms[1][r]), fmaxf(ms[2][r], ms[3][r]));
+            if (p.sink) M = fmaxf(M, p.sink[hbase + r]);
+            float L = p.sink ? expf(p.sink[hbase + r] - M) : 0.f;
+#pragma unroll
+            for (int w = 0; w < 4; ++w) {
+                f[w] = ms[w][r] == -INFINITY ? 0.f : expf(ms[w][r] - M);
+                L = fmaf(f[w], ls[w][r], L);
+            }
+            inv = 1.0f / L;
+        }
+        float u = 0.f, v = 0.f;
+#pragma unroll
+        for (int w = 0; w < 4; ++w) {
+            const float2 ov = *reinterpret_cast<const float2*>(Os + (w * kMdRows + r) * OS + col);
+            u = fmaf(f[w], ov.x, u);
+            v = fmaf(f[w], ov.y, v);
+        }
+        u *= inv;
+        v *= inv;
+        if (p.out_rot) {
+            const float u0 = u;
+            u = ma_unturn(p, row0, col, u0, v);
+            v = ma_unturn(p, row0, col + 1, v, u0);
+        }
+        const int64_t oc = (int64_t)(hbase + r) * vdim + col;
+        if (p.gate) {
+            u *= ma_gate<bf16_t>(p, row0, (int)oc);
+            v *= ma_gate<bf16_t>(p, row0, (int)oc + 1);
+        }
+        *reinterpret_cast<uint32_t*>(static_cast<bf16_t*>(p.out) + (int64_t)row0 * p.heads * vdim + oc) = pack_bf16x2(u, v);
+    }
+}
+
+template <int DIM, int VDIM, bool SHARED>
+static int md_launch(const MaskAttnParams& p, int ntiles, cudaStream_t st) {
+    const size_t tiles = ((size_t)md_stages(SHARED) * kMmKeys * (DIM + kMmPad) + (SHARED ? 0 : (size_t)md_stages(SHARED) * kMmKeys * (VDIM + kMmPad))) * sizeof(bf16_t);
+    const size_t merge = (size_t)4 * kMdRows * (VDIM + 4) * sizeof(float);
+    const size_t smem = (size_t)kMdRows * (DIM + kMmPad) * sizeof(bf16_t) + (tiles > merge ? tiles : merge);
+    auto kern = masked_attention_mma_decode_kernel<DIM, VDIM, SHARED>;
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+    const int hpg = p.heads / p.num_kv_heads;
+    dim3 grid((unsigned)ntiles, (unsigned)(p.num_kv_heads * ((hpg + kMdRows - 1) / kMdRows)));
+    kern<<<grid, kMmThreads, smem, st>>>(p);
+    PA_RETURN_LAUNCH_STATUS();
+}
+
+// PA_ERR_UNSUPPORTED: this shape or these pointers stay on the streaming kernel
+static int md_dispatch(const MaskAttnParams& p, int ntiles, cudaStream_t st) {
+    if (!mm_operands_ok(p)) return PA_ERR_UNSUPPORTED;
+    const int dp = mm_padded(p.dim), vp = mm_padded(p.vdim);
+    if (p.k_pool == p.v_pool) {
+#define PA_MD_CASE(D) if (dp == D) return md_launch<D, D, true>(p, ntiles, st)
+        PA_MD_CASE(32); PA_MD_CASE(64); PA_MD_CASE(128);
+#undef PA_MD_CASE
+        return PA_ERR_UNSUPPORTED;
+    }
+#define PA_MD_CASE(D, V) if (dp == D && vp == V) return md_launch<D, V, false>(p, ntiles, st)
+    PA_MD_CASE(32, 32); PA_MD_CASE(32, 64); PA_MD_CASE(32, 128);
+    PA_MD_CASE(64, 32); PA_MD_CASE(64, 64); PA_MD_CASE(64, 128);
+    PA_MD_CASE(128, 32); PA_MD_CASE(128, 64); PA_MD_CASE(128, 128);
+#undef PA_MD_CASE
     return PA_ERR_UNSUPPORTED;
 }
 
@@ -995,7 +1260,7 @@ PA_API int pa_masked_attention_gated(const void* d_q, int64_t q_stride, int q_of
     p.num_slots = num_slots; p.num_kv_heads = num_kv_heads; p.num_tiles = num_tiles; p.total_pages = total_pages;
     p.tile_size = tile_size; p.tiles = d_q_tiles; p.heads = heads; p.dim = dim; p.vdim = vdim; p.scale = scale;
     p.softcap = softcap; p.mask_kind = mask_kind; p.mask_size = mask_size; p.bias_kind = bias_kind; p.bias = d_bias;
-    p.bias_len = bias_len; p.out = d_out; p.head_rows = 0;
+    p.bias_len = bias_len; p.out = d_out;
     p.head_scale = d_head_scale; p.sink = d_sink; p.mask_keep = mask_keep; p.out_rot = d_out_rot;
     p.sigm = sigmoid_weights; p.key_scale = d_key_scale; p.head_bias = d_head_bias; p.gate = d_gate;
     p.gate_stride = gate_stride; p.gate_off = gate_off;
@@ -1004,6 +1269,8 @@ PA_API int pa_masked_attention_gated(const void* d_q, int64_t q_stride, int q_of
         if (elem != 2) return PA_ERR_UNSUPPORTED;
         return mm_dispatch(p, num_q_tiles, as_stream(stream));
     }
+    if (tile_kind == 3)         // every tile is one token: the heads of a kv head as rows on the tensor cores
+        return elem == 2 ? md_dispatch(p, num_q_tiles, as_stream(stream)) : PA_ERR_UNSUPPORTED;
     if (tile_kind == 1) {       // every tile is one token: the streaming kernel, where it serves the shape
         const int st = elem == 4 ? ma_decode_dispatch<float>(p, num_q_tiles, as_stream(stream))
                                  : ma_decode_dispatch<bf16_t>(p, num_q_tiles, as_stream(stream));

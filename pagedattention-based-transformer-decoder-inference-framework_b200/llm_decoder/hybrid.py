@@ -606,6 +606,9 @@ class MaskedAttention:
             if group is None:
                 continue
             tiles, ntiles, _longest = group
+            # decoded tokens of a batch with at least one (token, kv head) pair per SM: heads as rows on the tensor cores
+            if kind == 1 and mma_tokens and ntiles * self.kv_heads >= c.model.sm_count:
+                kind = 3
             st = lib.pa_masked_attention_gated(proj.data_ptr(), proj.stride(0), off, kv.key_buffer_.data_ptr(),
                                                values.data_ptr(), table.data_ptr(), pt.num_beams_, pt.num_heads_,
                                                pt.num_tiles_, kv.total_pages_, kv.tile_size_, tiles.data_ptr(), ntiles,
@@ -616,7 +619,7 @@ class MaskedAttention:
                                                _cabi.ptr(self.head_bias), _cabi.ptr(gate[0]),
                                                gate[0].stride(0) if gate[0] is not None else 0, gate[1], out.data_ptr(),
                                                c.elem, kind, s)
-            if kind == 2 and st == _cabi.PA_ERR_UNSUPPORTED:
+            if kind >= 2 and st == _cabi.PA_ERR_UNSUPPORTED:
                 return False
             _chk(st, "pa_masked_attention_gated")
         return True

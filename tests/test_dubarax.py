@@ -725,7 +725,7 @@ def test_attention_kernels_alone(heads, kv_heads, dim, vdim, mask, size, bias):
         tt = lib.pa_masked_attention_tile_tokens(heads, kv_heads)
         mt = lib.pa_masked_attention_mma_tile_tokens(dim, vdim, proj.element_size())
         table_dev = pt.device_data()
-        for use_mma, use_stream in ((0, 0), (mt, 1)):
+        for use_mma, single in ((0, 0), (mt, 1)) + (((mt, 3),) if mt else ()):      # 3: heads as rows on the tensor cores
             out = torch.zeros(sum(new), heads * vdim, dtype=dtype, device=dev)
             for kind, group in batch.query_tiles(tt, use_mma, 16).items():
                 if group is None:
@@ -735,7 +735,7 @@ def test_attention_kernels_alone(heads, kv_heads, dim, vdim, mask, size, bias):
                                              table_dev.data_ptr(), pt.num_beams_, pt.num_heads_, pt.num_tiles_, kv.total_pages_,
                                              kv.tile_size_, tiles.data_ptr(), ntiles, heads, dim, vdim, scale, cap, MASK_KIND[mask],
                                              size, bias_kind, _cabi.ptr(bias_t), int(bias_t.shape[0]) if bias_kind == 2 else 0,
-                                             out.data_ptr(), proj.element_size(), kind if (use_stream or kind != 1) else 0,
+                                             out.data_ptr(), proj.element_size(), single if kind == 1 else kind,
                                              _cabi.stream())
                 assert rc == 0, (kind, rc)
             err = (out.double().cpu() - want).abs().max().item()

@@ -625,7 +625,7 @@ def test_attention_kernels_alone(heads, kv_heads, dim, vdim, mask, size, keep, s
         mt = lib.pa_masked_attention_mma_tile_tokens(dim, vdim, proj.element_size())
         table_dev = pt.device_data()
         td, sd = (temps.to(dev) if temp else None), (sinks.to(dev) if sinks is not None else None)
-        for use_mma, use_stream in ((0, 0), (mt, 1)):
+        for use_mma, single in ((0, 0), (mt, 1)) + (((mt, 3),) if mt else ()):      # 3: heads as rows on the tensor cores
             out = torch.zeros(sum(new), heads * vdim, dtype=dtype, device=dev)
             for kind, group in batch.query_tiles(tt, use_mma, 16).items():
                 if group is None:
@@ -636,7 +636,7 @@ def test_attention_kernels_alone(heads, kv_heads, dim, vdim, mask, size, keep, s
                                                   pt.num_tiles_, kv.total_pages_, kv.tile_size_, tiles.data_ptr(), ntiles, heads, dim,
                                                   vdim, scale, 0.0, MASK_KIND[mask], size, keep if mask == "window" else 0, 0, None, 0,
                                                   _cabi.ptr(td), _cabi.ptr(sd), _cabi.ptr(rot), out.data_ptr(), proj.element_size(),
-                                                  kind if (use_stream or kind != 1) else 0, _cabi.stream())
+                                                  single if kind == 1 else kind, _cabi.stream())
                 assert rc == 0, (kind, rc)
             err = (out.double().cpu() - want).abs().max().item()
             assert err < tol * max(1.0, want.abs().max().item()), (dtype, use_mma, err)

@@ -287,6 +287,26 @@ def test_mixed_batches_of_unequal_requests(name, dtype):
 
 
 @pytest.mark.gpu
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_large_decode_batch(dtype):
+    """80 sequences of unequal length decode two tokens side by side: enough (token, key/value head) pairs for the
+    tensor-core kernel of decoded tokens, windows of one key up to the whole sequence."""
+    import llm_decoder as ld
+    config = R.make_config([R.window_layer(heads=6, kv_heads=2, dim=16, size=21), R.latent_layer(heads=3, dim=8, rot_dim=8, kv_rank=16),
+                            R.window_layer(heads=4, kv_heads=2, dim=40, size=70, ff=None), R.retention_layer(heads=2, dim=8, vdim=8, rot_dims=8)],
+                           width=64, streams=2)
+    W = R.random_weights(config, 11)
+    lens = [1 + (i * 7) % 90 for i in range(80)]
+    seqs = [_tokens(n + 2, config["vocab"], 500 + i) for i, n in enumerate(lens)]
+    eng = ld.Engine(_model(config, W, dtype, max_tokens=80 * 96, max_seqs=80))
+    eng.step([(i, q[:-2], []) for i, q in enumerate(seqs)])
+    got = [eng.step([(i, q[t:t + 1] if t + 1 else q[t:], [0]) for i, q in enumerate(seqs)]) for t in (-2, -1)]
+    want = [R.forward(config, W, q)[-2:] for q in seqs]
+    for t in (0, 1):
+        _close(got[t], torch.stack([w[t] for w in want]), dtype)
+
+
+@pytest.mark.gpu
 def test_wanted_rows_and_steps_without_any():
     """Logits of some rows, in any order and twice, and steps in which nothing is wanted (their cache and state stay)."""
     import llm_decoder as ld
@@ -639,7 +659,8 @@ def test_attention_kernels_alone(heads, kv_heads, dim, weights, shared, gate, bi
         mt = lib.pa_masked_attention_mma_tile_tokens(dim, dim, proj.element_size())
         hbd = hb.to(dev)
         vals = kv.key_buffer_ if shared else kv.value_buffer_
-        for use_mma, use_stream in ((0, 0), (mt, 1)):
+        # single tokens: the tile kernel, the streaming kernel, and (where the shape is served) heads as rows on the tensor cores
+        for use_mma, single in ((0, 0), (mt, 1)) + (((mt, 3),) if mt else ()):
             out = torch.zeros(sum(new), qc, dtype=dtype, device=dev)
             for kind, group in batch.query_tiles(tt, use_mma, 16).items():
                 if group is None:
@@ -650,7 +671,7 @@ def test_attention_kernels_alone(heads, kv_heads, dim, weights, shared, gate, bi
                                    heads, dim, dim, scale, 0.0, 1, size, 0, 0, None, 0, None, None, None, _cabi.ptr(kv.key_scale_),
                                    1 if weights == "sigmoid" else 0, hbd.data_ptr() if bias else None, proj.data_ptr() if gate else None,
                                    proj.stride(0), cols - qc, out.data_ptr(), proj.element_size(), kd, s)
-                rc = lib.pa_masked_attention_gated(*args(kind if (use_stream or kind != 1) else 0))
+                rc = lib.pa_masked_attention_gated(*args(single if kind == 1 else kind))
                 assert rc == 0, (kind, rc)
             err = (out.double().cpu() - want).abs().max().item()
             assert err < tol * max(1.0, want.abs().max().item()), (dtype, use_mma, err)
