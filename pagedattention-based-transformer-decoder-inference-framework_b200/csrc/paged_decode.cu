@@ -642,8 +642,7 @@ __global__ void __launch_bounds__(NW * 32, 1) paged_decode_overlap_kernel(const 
 
     auto produce = [&]() {
         if (!p_has) return;
-        // elect.sync, not `lane == 0`: the bulk copies keep their operands in uniform registers and are issued
-        // back to back (under lane == 0 the compiler cannot prove them warp-uniform and serialises the issue)
+        // elect.sync, not `lane == 0`: the bulk copies are issued back to back (measurably slower under lane == 0)
         if (elect_one()) {
             const int nvalid = (p_page >= 0) ? min(kUnitTok, p_rem) : 0;
             my_meta[p_st] = nvalid;
