@@ -865,6 +865,54 @@ int pa_streams_add_norm(const float* d_src, int src_streams, float* d_dst, int64
                         const float* d_gain, float* d_u, void* d_next, const int32_t* d_row_ids, int elem,
                         pa_stream_t stream);
 
+/* ---- token-pair embedding, block passes that add, convolved + turned + normed projections, sinks on the latent ---------
+ * pa_embedding_bigram: x[r] = embed[ids[r]] * scale + bigram[b(r)] as float (tables in the activation type), b(r) =
+ *   (prev_ids[r] * mul_prev + ids[r] * mul_cur) mod buckets, or row `buckets` (the table has buckets + 1 rows) where
+ *   prev_ids[r] is -1 (the first token of a sequence); out-of-range ids give zeros.  d_copy (NULL: none): the same rows again.
+ * pa_residual_add_norm2_pass: pa_residual_add_norm2 where, after the addends, x[r] += d_base[r] and x[r] += d_step (float
+ *   rows, each optional) come before the norms.
+ * pa_rope_table_scaled: pa_rope_table for the angles d_row_pos[r] * d_freqs[i] (double, [dims / 2]); cos and sin * mult.
+ * pa_latent_turn_append: pa_latent_norm_append where, in the same launch, the queries of the rows are rotated in place:
+ *   pairs of the first rot_dims columns from q_off + h * q_head_stride of row r of d_q, h < heads.
+ * pa_gate_rows: out[r, c] = in[r, c] * sigmoid(gate[r, c]); out may be in.
+ * pa_latent_attention_sink: pa_latent_attention where exp(d_sink[h]) (NULL: none) joins head h's softmax denominator once.
+ * pa_conv_rope_norm_append: everything between the input product and the attention of a layer in one launch.  The raw rows
+ *   hold q | k | v from column in_off; every channel passes the causal convolution of `taps` taps (d_weight [taps][channels],
+ *   entry b = the weight b tokens back; NULL: none) whose last taps - 1 raw rows are kept in d_state [slots][taps - 1]
+ *   [channels] (oldest first, updated here); queries and keys are rotated over their first rot_dims dimensions
+ *   (neighbouring pairs, d_rope [rows][rot_dims / 2][cos, sin]) and, with norm 1, divided by sqrt(mean square over dim + eps),
+ *   all in float.  Queries go to d_q_out (not d_in), keys and values to the pools (NULL: a layer that reads another
+ *   layer's pool; the rows then hold queries only).  d_items [num_items][6] = first row, tokens (at most item_tokens, at
+ *   least taps - 1 of which the portion's earlier items hold each), slot, offset within the portion, the portion's length,
+ *   first position.  At most 8 taps, heads of at most 512. */
+int pa_embedding_bigram(const void* d_embed, const void* d_bigram, int elem, const int32_t* d_ids, const int32_t* d_prev_ids,
+                        int rows, int width, int vocab, int64_t buckets, int64_t mul_prev, int64_t mul_cur, float scale,
+                        float* d_out, float* d_copy, pa_stream_t stream);
+int pa_residual_add_norm2_pass(float* d_x, int64_t rows, int width, const void* d_y, const void* d_y2, const float* d_routed,
+                               const float* d_sel_w, const int32_t* d_sel_id, int top, int experts, const void* d_ident,
+                               const float* d_base, const float* d_step, float eps, const float* d_gain1, void* d_next1,
+                               const float* d_gain2, void* d_next2, int elem, pa_stream_t stream);
+int pa_rope_table_scaled(const int32_t* d_row_pos, int rows, int dims, const double* d_freqs, double mult, float* d_table,
+                         pa_stream_t stream);
+int pa_latent_turn_append(void* d_pool, const int32_t* d_table, int num_slots, int num_tiles, int total_pages, int tile_size,
+                          int kv_rank, int rot_dim, int rot_dims, int pairing, const void* d_src, int64_t src_stride, int c_off,
+                          const float* d_gain, float eps, const float* d_rope_table, void* d_q, int64_t q_stride, int q_off,
+                          int heads, int q_head_stride, const int32_t* d_row_slot, const int32_t* d_row_pos, int rows, int elem,
+                          pa_stream_t stream);
+int pa_gate_rows(const void* d_in, int64_t in_stride, const void* d_gate, int64_t gate_stride, int cols, int64_t rows,
+                 void* d_out, int64_t out_stride, int elem, pa_stream_t stream);
+int pa_latent_attention_sink(const void* d_q_lat, int64_t ql_row_stride, int64_t ql_head_stride, const void* d_q_rot,
+                             int64_t qr_row_stride, int64_t qr_head_stride, const void* d_pool, const int32_t* d_table,
+                             int num_slots, int num_tiles, int total_pages, int tile_size, const int32_t* d_q_tiles,
+                             int num_q_tiles, int heads, int kv_rank, int rot_dim, float scale, const float* d_sink,
+                             void* d_out, int64_t o_row_stride, int64_t o_head_stride, int elem, int nsplit, int tile_kind,
+                             void* d_workspace, size_t workspace_bytes, pa_stream_t stream);
+int pa_conv_rope_norm_append(const void* d_in, int64_t in_stride, int in_off, int heads, int kv_heads, int dim, int vdim,
+                             int taps, const float* d_weight, float* d_state, int rot_dims, const float* d_rope, int norm,
+                             float eps, void* d_q_out, int64_t q_out_stride, void* d_k_pool, void* d_v_pool,
+                             const int32_t* d_table, int num_slots, int num_tiles, int total_pages, int tile_size,
+                             const int32_t* d_items, int num_items, int item_tokens, int elem, pa_stream_t stream);
+
 #ifdef __cplusplus
 }
 #endif

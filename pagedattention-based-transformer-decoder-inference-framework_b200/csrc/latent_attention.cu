@@ -11,17 +11,21 @@
 // so attention is multi-query attention of the `heads` latent queries ql_h = Wuk_h^T qp_h (kv_rank wide, next to the
 // rotated part) against the pool rows, whose first kv_rank columns are also the values; Wuk^T before and Wuv after are
 // per-head matrix products over the batch rows (head_linear_kernel).  Scores, softmax weights and the weighted sums are
-// float; pool rows are stored in the activation type (float or bfloat16).
+// float; pool rows are stored in the activation type (float or bfloat16).  With sinks, exp(sink_h) joins the softmax
+// denominator of head h once (a logit without key or value).
 //
 //   rope_table_kernel        cos / sin of p * base^(-2i / dims) per batch row (angles in double, table in float)
+//   rope_table_scaled_kernel the same for given frequencies, times a factor (stretched rotations)
 //   rope_rows_kernel         in-place rotation of the pairs of every head's rotated part: (2i, 2i + 1), or halves
 //                            (i, i + dims / 2)
 //   latent_kv_append_kernel  RMS norm (per-channel gain) of the latent columns + rotation of the shared key part, written
-//                            to the row's place in the pool; optionally the norm of the query latent in the same launch
+//                            to the row's place in the pool; optionally the norm of the query latent, or the rotation of
+//                            all heads' queries in place, in the same launch
 //   head_linear_kernel       out[r, h, :] = x[r, h, :] . W[h]  (W [heads][K][N]), any strides
 //   latent_attention_kernel  float tile kernel, any shape, keys optionally split with a merge kernel
 //   latent_attention_mma_kernel  bfloat16 tensor-core kernel (mma.sync), see there
 //   head_gate_kernel         out[r, h * vdim + v] = in[r, h, v] * sigmoid(gate[r, h])
+//   gate_rows_kernel         out[r, c] = in[r, c] * sigmoid(gate[r, c])
 #include "seq_common.cuh"
 
 namespace pa {
@@ -38,6 +42,17 @@ __global__ void rope_table_kernel(const int32_t* __restrict__ row_pos, int rows,
     sincos(a, &s, &c);
     table[2 * i] = (float)c;
     table[2 * i + 1] = (float)s;
+}
+
+// the same with the angle per position of every pair given (double), cos and sin multiplied by mult
+__global__ void rope_table_scaled_kernel(const int32_t* __restrict__ row_pos, int rows, int half,
+                                         const double* __restrict__ freqs, double mult, float* __restrict__ table) {
+    const int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= (int64_t)rows * half) return;
+    double s, c;
+    sincos((double)row_pos[i / half] * freqs[i % half], &s, &c);
+    table[2 * i] = (float)(c * mult);
+    table[2 * i + 1] = (float)(s * mult);
 }
 
 // the two members of pair k of `half` pairs: neighbours (pairing 0) or entry k of either half (pairing 1)
@@ -78,19 +93,35 @@ __device__ __forceinline__ void rms_row_warp(const T* __restrict__ s, int width,
 }
 
 // One warp per (row, unit): src row = [.. | c_raw (kv_rank) at c_off | kr_raw (rot_dim) right behind it]; unit 0 appends
-// it, unit 1 (units == 2) norms the query latent of the same row: q_rank columns at q_off -> q_out.
+// it; unit 1 (units == 2) either norms the query latent of the same row, q_rank columns at q_off -> q_out, or (turn_q)
+// rotates the row's queries in place: pairs k < rot_dims / 2 from column q_off + h * q_head_stride of q_out, h < heads.
 template <typename T>
 __global__ void latent_kv_append_kernel(T* __restrict__ pool, const int32_t* __restrict__ table, int num_slots,
                                         int num_tiles, int total_pages, int tile_size, int kv_rank, int rot_dim,
-                                        int rot_dims, const T* __restrict__ src, int64_t src_stride, int c_off,
+                                        int rot_dims, const T* src, int64_t src_stride, int c_off,
                                         const float* __restrict__ gain, float eps, const float* __restrict__ rope,
                                         const int32_t* __restrict__ row_slot, const int32_t* __restrict__ row_pos,
                                         int rows, int pairing, int units, int q_off, int q_rank,
-                                        const float* __restrict__ q_gain, T* __restrict__ q_out, int64_t q_out_stride) {
+                                        const float* __restrict__ q_gain, T* q_out, int64_t q_out_stride,
+                                        int turn_q, int heads, int q_head_stride) {
     const int lane = threadIdx.x & 31;
     const int64_t w = ((int64_t)blockIdx.x * blockDim.x + threadIdx.x) >> 5;
     if (w >= (int64_t)rows * units) return;
     const int64_t r = w / units;
+    if (w % units == 1 && turn_q) {
+        const int half = rot_dims / 2;
+        T* q = q_out + r * q_out_stride + q_off;
+        for (int i = lane; i < heads * half; i += 32) {
+            const int k = i % half;
+            const float2 t = *reinterpret_cast<const float2*>(rope + (r * half + k) * 2);
+            T* p0 = q + (int64_t)(i / half) * q_head_stride + pair_first(k, pairing);
+            T* p1 = q + (int64_t)(i / half) * q_head_stride + pair_second(k, half, pairing);
+            const float u = to_f32<T>(*p0), v = to_f32<T>(*p1);
+            *p0 = from_f32<T>(u * t.x - v * t.y);
+            *p1 = from_f32<T>(v * t.x + u * t.y);
+        }
+        return;
+    }
     if (w % units == 1) {
         rms_row_warp<T>(src + r * src_stride + q_off, q_rank, eps, q_gain, q_out + r * q_out_stride, lane);
         return;
@@ -204,6 +235,25 @@ __global__ void head_gate_bf16x8_kernel(const bf16_t* __restrict__ in, int64_t i
     *reinterpret_cast<uint4*>(out + i) = bf16x8_pack(f);
 }
 
+// out[r, c] = in[r, c] * sigmoid(gate[r, c]), one CTA per row; out may be in.  VEC 8: bfloat16 rows in 16-byte words
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256) gate_rows_kernel(const T* in, int64_t i_rs, const T* __restrict__ gate, int64_t g_rs,
+                                                        int cols, T* out, int64_t o_rs) {
+    const int64_t r = blockIdx.x;
+    for (int c = threadIdx.x * VEC; c < cols; c += blockDim.x * VEC) {
+        if constexpr (VEC == 8) {
+            float f[8], g[8];
+            bf16x8_unpack(*reinterpret_cast<const uint4*>(in + r * i_rs + c), f);
+            bf16x8_unpack(*reinterpret_cast<const uint4*>(gate + r * g_rs + c), g);
+#pragma unroll
+            for (int k = 0; k < 8; ++k) f[k] *= sigmoid_f32(g[k]);
+            *reinterpret_cast<uint4*>(out + r * o_rs + c) = bf16x8_pack(f);
+        } else {
+            out[r * o_rs + c] = from_f32<T>(to_f32<T>(in[r * i_rs + c]) * sigmoid_f32(to_f32<T>(gate[r * g_rs + c])));
+        }
+    }
+}
+
 // ---- attention: float tile kernel -----------------------------------------------------------------------------------
 constexpr int kLaRows = 32;     // (token, head) rows per CTA
 constexpr int kLaWarps = 8;
@@ -226,7 +276,18 @@ struct LatentAttnParams {
     int nsplit;
     float* partial;             // nsplit > 1: [(tile, chunk, split, row)][2 + kv_rank], m in natural-log units
     int cta_rows;               // (token, head) rows per CTA: kLaRows (float kernel) or kLmRows (tensor-core kernel)
+    const float* sink;          // [heads] or null
 };
+
+// The factor of head h's accumulated sums: 1 / denominator.  m: the reference the sums were taken at (natural-log units).
+// A sink far above m takes the reference over, so nothing overflows.
+__device__ __forceinline__ float la_inv_sum(const LatentAttnParams& p, int h, float m, float l) {
+    if (!p.sink) return 1.0f / l;
+    const float sk = p.sink[h];
+    if (sk <= m) return 1.0f / (l + expf(sk - m));
+    const float c = expf(m - sk);
+    return c / fmaf(l, c, 1.0f);
+}
 
 __host__ __device__ __forceinline__ void la_geometry(int heads, int cta_rows, int& hc, int& nchunk) {
     hc = heads < cta_rows ? heads : cta_rows;
@@ -355,7 +416,7 @@ __global__ void __launch_bounds__(kLaWarps * 32) latent_attention_kernel(const L
         } else if (rpos[r] >= 0) {
             const int tok = row / hc, hh = chunk * hc + row % hc;
             T* dst = static_cast<T*>(p.out) + (int64_t)(row0 + tok) * p.o_rs + (int64_t)hh * p.o_hs;
-            const float inv = 1.0f / l[r];
+            const float inv = la_inv_sum(p, hh, m[r], l[r]);
 #pragma unroll
             for (int i = 0; i < NV; ++i)
                 if (lane + 32 * i < p.kv_rank) dst[lane + 32 * i] = from_f32<T>(acc[r][i] * inv);
@@ -391,7 +452,7 @@ __global__ void __launch_bounds__(kLaWarps * 32) latent_attention_merge_kernel(c
                 if (lane + 32 * i < p.kv_rank) acc[i] = fmaf(w, pz[2 + lane + 32 * i], acc[i]);
         }
         T* dst = static_cast<T*>(p.out) + (int64_t)(row0 + tok) * p.o_rs + (int64_t)hh * p.o_hs;
-        const float inv = 1.0f / l;
+        const float inv = la_inv_sum(p, hh, M, l);
 #pragma unroll
         for (int i = 0; i < NV; ++i)
             if (lane + 32 * i < p.kv_rank) dst[lane + 32 * i] = from_f32<T>(acc[i] * inv);
@@ -761,7 +822,7 @@ __global__ void __launch_bounds__(kLmThreads, 1) latent_attention_mma_kernel(con
                 if (col < kv_rank) { dst[2 + col] = o[t][2 * i]; dst[2 + col + 1] = o[t][2 * i + 1]; }
             }
         } else {
-            const float inv = 1.0f / l[i];
+            const float inv = la_inv_sum(p, hh, m[i] * 0.6931471805599453f, l[i]);
             bf16_t* dst = static_cast<bf16_t*>(p.out) + (int64_t)(row0 + tok) * p.o_rs + (int64_t)hh * p.o_hs;
 #pragma unroll
             for (int t = 0; t < NT; ++t) {
@@ -830,11 +891,40 @@ static int lm_dispatch(const LatentAttnParams& p, int ntiles, bool one_token_til
 
 using namespace pa;
 
+static int latent_append(void* d_pool, const int32_t* d_table, int num_slots, int num_tiles, int total_pages, int tile_size,
+                         int kv_rank, int rot_dim, int rot_dims, int pairing, const void* d_src, int64_t src_stride, int c_off,
+                         const float* d_gain, float eps, const float* d_rope_table, int q_off, int q_rank,
+                         const float* d_q_gain, void* d_q_out, int64_t q_out_stride, int turn_q, int heads, int q_head_stride,
+                         const int32_t* d_row_slot, const int32_t* d_row_pos, int rows, int elem, pa_stream_t stream) {
+    PA_CHECK_ARG(d_pool && d_table && d_src && d_gain && d_row_slot && d_row_pos && rows >= 0 && (pairing == 0 || pairing == 1));
+    PA_CHECK_ARG(num_slots > 0 && num_tiles > 0 && total_pages > 0 && tile_size > 0 && kv_rank > 0 && rot_dim >= 0);
+    PA_CHECK_ARG(rot_dims >= 0 && rot_dims <= rot_dim && rot_dims % 2 == 0 && (rot_dims == 0 || d_rope_table));
+    if (rows == 0) return PA_OK;
+    const int units = d_q_out ? 2 : 1;
+    const int64_t threads = (int64_t)rows * units * 32;
+    PA_DISPATCH_ELEM(elem, latent_kv_append_kernel<T><<<(unsigned)((threads + 255) / 256), 256, 0, as_stream(stream)>>>(
+                               static_cast<T*>(d_pool), d_table, num_slots, num_tiles, total_pages, tile_size, kv_rank,
+                               rot_dim, rot_dims, static_cast<const T*>(d_src), src_stride, c_off, d_gain, eps,
+                               d_rope_table, d_row_slot, d_row_pos, rows, pairing, units, q_off, q_rank, d_q_gain,
+                               static_cast<T*>(d_q_out), q_out_stride, turn_q, heads, q_head_stride));
+    PA_RETURN_LAUNCH_STATUS();
+}
+
 PA_API int pa_rope_table(const int32_t* d_row_pos, int rows, int dims, float base, float* d_table, pa_stream_t stream) {
     PA_CHECK_ARG(d_row_pos && d_table && rows >= 0 && dims >= 0 && dims % 2 == 0 && base > 0.f);
     const int64_t n = (int64_t)rows * (dims / 2);
     if (n == 0) return PA_OK;
     rope_table_kernel<<<(unsigned)((n + 127) / 128), 128, 0, as_stream(stream)>>>(d_row_pos, rows, dims, log((double)base), d_table);
+    PA_RETURN_LAUNCH_STATUS();
+}
+
+PA_API int pa_rope_table_scaled(const int32_t* d_row_pos, int rows, int dims, const double* d_freqs, double mult,
+                                float* d_table, pa_stream_t stream) {
+    PA_CHECK_ARG(d_row_pos && d_freqs && d_table && rows >= 0 && dims >= 0 && dims % 2 == 0);
+    const int64_t n = (int64_t)rows * (dims / 2);
+    if (n == 0) return PA_OK;
+    rope_table_scaled_kernel<<<(unsigned)((n + 127) / 128), 128, 0, as_stream(stream)>>>(d_row_pos, rows, dims / 2, d_freqs, mult,
+                                                                                        d_table);
     PA_RETURN_LAUNCH_STATUS();
 }
 
@@ -869,19 +959,22 @@ PA_API int pa_latent_norm_append(void* d_pool, const int32_t* d_table, int num_s
                                  int q_off, int q_rank, const float* d_q_gain, void* d_q_out, int64_t q_out_stride,
                                  const int32_t* d_row_slot, const int32_t* d_row_pos, int rows, int elem,
                                  pa_stream_t stream) {
-    PA_CHECK_ARG(d_pool && d_table && d_src && d_gain && d_row_slot && d_row_pos && rows >= 0);
-    PA_CHECK_ARG((pairing == 0 || pairing == 1) && (!d_q_out || (d_q_gain && q_rank > 0)));
-    PA_CHECK_ARG(num_slots > 0 && num_tiles > 0 && total_pages > 0 && tile_size > 0 && kv_rank > 0 && rot_dim >= 0);
-    PA_CHECK_ARG(rot_dims >= 0 && rot_dims <= rot_dim && rot_dims % 2 == 0 && (rot_dims == 0 || d_rope_table));
-    if (rows == 0) return PA_OK;
-    const int units = d_q_out ? 2 : 1;
-    const int64_t threads = (int64_t)rows * units * 32;
-    PA_DISPATCH_ELEM(elem, latent_kv_append_kernel<T><<<(unsigned)((threads + 255) / 256), 256, 0, as_stream(stream)>>>(
-                               static_cast<T*>(d_pool), d_table, num_slots, num_tiles, total_pages, tile_size, kv_rank,
-                               rot_dim, rot_dims, static_cast<const T*>(d_src), src_stride, c_off, d_gain, eps,
-                               d_rope_table, d_row_slot, d_row_pos, rows, pairing, units, q_off, q_rank, d_q_gain,
-                               static_cast<T*>(d_q_out), q_out_stride));
-    PA_RETURN_LAUNCH_STATUS();
+    PA_CHECK_ARG(!d_q_out || (d_q_gain && q_rank > 0));
+    return latent_append(d_pool, d_table, num_slots, num_tiles, total_pages, tile_size, kv_rank, rot_dim, rot_dims, pairing, d_src,
+                         src_stride, c_off, d_gain, eps, d_rope_table, q_off, q_rank, d_q_gain, d_q_out, q_out_stride, 0, 0, 0,
+                         d_row_slot, d_row_pos, rows, elem, stream);
+}
+
+PA_API int pa_latent_turn_append(void* d_pool, const int32_t* d_table, int num_slots, int num_tiles, int total_pages,
+                                 int tile_size, int kv_rank, int rot_dim, int rot_dims, int pairing, const void* d_src,
+                                 int64_t src_stride, int c_off, const float* d_gain, float eps, const float* d_rope_table,
+                                 void* d_q, int64_t q_stride, int q_off, int heads, int q_head_stride,
+                                 const int32_t* d_row_slot, const int32_t* d_row_pos, int rows, int elem,
+                                 pa_stream_t stream) {
+    PA_CHECK_ARG(d_q && heads > 0 && q_head_stride >= rot_dims && q_off >= 0);
+    return latent_append(d_pool, d_table, num_slots, num_tiles, total_pages, tile_size, kv_rank, rot_dim, rot_dims, pairing, d_src,
+                         src_stride, c_off, d_gain, eps, d_rope_table, q_off, 0, nullptr, rot_dims ? d_q : nullptr, q_stride, 1,
+                         heads, q_head_stride, d_row_slot, d_row_pos, rows, elem, stream);
 }
 
 PA_API int pa_rms_norm_rows(const void* d_src, int64_t src_stride, int off, int width, float eps, const float* d_gain,
@@ -926,6 +1019,23 @@ PA_API int pa_head_gate(const void* d_in, int64_t in_row_stride, int64_t in_head
     PA_RETURN_LAUNCH_STATUS();
 }
 
+PA_API int pa_gate_rows(const void* d_in, int64_t in_stride, const void* d_gate, int64_t gate_stride, int cols, int64_t rows,
+                        void* d_out, int64_t out_stride, int elem, pa_stream_t stream) {
+    PA_CHECK_ARG(d_in && d_gate && d_out && cols > 0 && rows >= 0);
+    if (rows == 0) return PA_OK;
+    if (elem == 2 && cols % 8 == 0 && in_stride % 8 == 0 && gate_stride % 8 == 0 && out_stride % 8 == 0 &&
+        ((uintptr_t)d_in | (uintptr_t)d_gate | (uintptr_t)d_out) % 16 == 0) {
+        gate_rows_kernel<bf16_t, 8><<<(unsigned)rows, 256, 0, as_stream(stream)>>>(
+            static_cast<const bf16_t*>(d_in), in_stride, static_cast<const bf16_t*>(d_gate), gate_stride, cols,
+            static_cast<bf16_t*>(d_out), out_stride);
+        PA_RETURN_LAUNCH_STATUS();
+    }
+    PA_DISPATCH_ELEM(elem, gate_rows_kernel<T, 1><<<(unsigned)rows, 256, 0, as_stream(stream)>>>(
+                               static_cast<const T*>(d_in), in_stride, static_cast<const T*>(d_gate), gate_stride, cols,
+                               static_cast<T*>(d_out), out_stride));
+    PA_RETURN_LAUNCH_STATUS();
+}
+
 PA_API int pa_latent_attention_tile_tokens(int heads) {
     if (heads <= 0) return 0;
     return kLaRows / (heads < kLaRows ? heads : kLaRows);
@@ -950,6 +1060,18 @@ PA_API int pa_latent_attention(const void* d_q_lat, int64_t ql_row_stride, int64
                                int num_q_tiles, int heads, int kv_rank, int rot_dim, float scale, void* d_out,
                                int64_t o_row_stride, int64_t o_head_stride, int elem, int nsplit, int tile_kind,
                                void* d_workspace, size_t workspace_bytes, pa_stream_t stream) {
+    return pa_latent_attention_sink(d_q_lat, ql_row_stride, ql_head_stride, d_q_rot, qr_row_stride, qr_head_stride, d_pool, d_table,
+                                    num_slots, num_tiles, total_pages, tile_size, d_q_tiles, num_q_tiles, heads, kv_rank, rot_dim,
+                                    scale, nullptr, d_out, o_row_stride, o_head_stride, elem, nsplit, tile_kind, d_workspace,
+                                    workspace_bytes, stream);
+}
+
+PA_API int pa_latent_attention_sink(const void* d_q_lat, int64_t ql_row_stride, int64_t ql_head_stride, const void* d_q_rot,
+                                    int64_t qr_row_stride, int64_t qr_head_stride, const void* d_pool, const int32_t* d_table,
+                                    int num_slots, int num_tiles, int total_pages, int tile_size, const int32_t* d_q_tiles,
+                                    int num_q_tiles, int heads, int kv_rank, int rot_dim, float scale, const float* d_sink,
+                                    void* d_out, int64_t o_row_stride, int64_t o_head_stride, int elem, int nsplit,
+                                    int tile_kind, void* d_workspace, size_t workspace_bytes, pa_stream_t stream) {
     PA_CHECK_ARG(d_q_lat && (d_q_rot || rot_dim == 0) && d_pool && d_table && d_q_tiles && d_out && num_q_tiles >= 0);
     PA_CHECK_ARG(num_slots > 0 && num_tiles > 0 && total_pages > 0 && tile_size > 0 && heads > 0 && kv_rank > 0 && rot_dim >= 0);
     if (num_q_tiles == 0) return PA_OK;
@@ -963,6 +1085,7 @@ PA_API int pa_latent_attention(const void* d_q_lat, int64_t ql_row_stride, int64
     p.tile_size = tile_size; p.tiles = d_q_tiles; p.heads = heads; p.kv_rank = kv_rank; p.rot_dim = rot_dim; p.scale = scale;
     p.out = d_out; p.o_rs = o_row_stride; p.o_hs = o_head_stride; p.nsplit = nsplit; p.partial = static_cast<float*>(d_workspace);
     p.cta_rows = tile_kind >= 2 ? kLmRows : kLaRows;
+    p.sink = d_sink;
     if (elem != 4 && elem != 2) return PA_ERR_UNSUPPORTED;
     if (tile_kind == 2 || tile_kind == 3)
         return elem == 2 ? lm_dispatch(p, num_q_tiles, tile_kind == 3, as_stream(stream)) : PA_ERR_UNSUPPORTED;

@@ -141,6 +141,220 @@ __global__ void __launch_bounds__(256) qk_norm_kv_append_kernel(T* __restrict__ 
     }
 }
 
+// ---- short convolution, rotation and norm of this step's q | k | v rows fused with the append -----------------------------
+// One warp per (work item, unit): an item is a run of consecutive tokens of one portion, units are the query heads, the key
+// heads and the value heads (the latter two only where the layer has a pool of its own).  Per token and channel
+//     y_t = sum_b w[b] u_(t - b)      (b tokens back; w == null: y_t = u_t)
+// over the RAW projected rows u (before the portion: the state slot's last taps - 1 rows), accumulated in float; queries and
+// keys are then rotated over their first rot_dims dimensions (neighbouring pairs) and, with `norm`, divided by their root
+// mean square over dim -- both still in float, one rounding at the end.  Queries go to q_out, keys and values to their place
+// in the pools.  A lane owns the pairs (2 lane + 64 i, + 1) and slides a window of inputs along the item, so every raw row
+// is read once per item (plus the taps - 1 rows before it).  The items that START a portion leave the state for the next
+// step: they are the only readers of the slot's old rows, channel by channel in the same thread.
+struct ConvAppendParams {
+    const void* in;             // raw rows [q | k | v] from column in_off
+    int64_t in_stride;
+    int in_off, channels, heads, kv_heads, dim, vdim, rot_dims, taps;
+    const float* w;             // [taps][channels], entry b = the weight b tokens back, or null
+    float* state;               // [slots][taps - 1][channels], oldest row first
+    const float* rope;          // [rows][rot_dims / 2][cos, sin] of the batch rows
+    int norm;
+    float eps;
+    void* q_out;
+    int64_t q_out_stride;
+    void* k_pool;
+    void* v_pool;
+    const int32_t* table;
+    int num_slots, num_tiles, total_pages, tile_size;
+    const int32_t* items;       // [n][6]: first row, tokens, slot, offset within the portion, portion's length, first position
+    int num_items;
+    int pairs;                  // every pair of columns starts on a boundary of two elements
+};
+constexpr int kCaMaxTaps = 8;
+
+template <typename T>
+__device__ __forceinline__ void ca_load(const T* __restrict__ p, int pairs, bool second, float& u, float& v) {
+    if (pairs) {
+        if constexpr (sizeof(T) == 2) {
+            const uint32_t w = *reinterpret_cast<const uint32_t*>(p);
+            u = __uint_as_float(w << 16);
+            v = __uint_as_float(w & 0xffff0000u);
+        } else {
+            const float2 w = *reinterpret_cast<const float2*>(p);
+            u = w.x;
+            v = w.y;
+        }
+    } else {
+        u = to_f32<T>(p[0]);
+        v = second ? to_f32<T>(p[1]) : 0.f;
+    }
+}
+template <typename T>
+__device__ __forceinline__ void ca_store(T* __restrict__ p, int pairs, bool second, float u, float v) {
+    if (pairs) {
+        if constexpr (sizeof(T) == 2) *reinterpret_cast<uint32_t*>(p) = pack_bf16x2(u, v);
+        else *reinterpret_cast<float2*>(p) = make_float2(u, v);
+    } else {
+        p[0] = from_f32<T>(u);
+        if (second) p[1] = from_f32<T>(v);
+    }
+}
+
+// NP: pairs per lane; TAPS: padded taps (the weights past `taps` are zero)
+template <typename T, int NP, int TAPS>
+__global__ void __launch_bounds__(256) conv_rope_norm_append_kernel(const ConvAppendParams p) {
+    const int lane = threadIdx.x & 31;
+    const int units = p.heads + (p.k_pool ? 2 * p.kv_heads : 0);
+    const int64_t wid = ((int64_t)blockIdx.x * blockDim.x + threadIdx.x) >> 5;
+    if (wid >= (int64_t)p.num_items * units) return;
+    const int unit = (int)(wid % units);
+    const int* it = p.items + 6 * (wid / units);
+    const int row0 = it[0], n = it[1], slot = it[2], off = it[3], plen = it[4], pos0 = it[5];
+    if ((unsigned)slot >= (unsigned)p.num_slots) return;
+    const int kind = unit < p.heads ? 0 : unit < p.heads + p.kv_heads ? 1 : 2;       // query, key, value
+    const int g = kind == 0 ? 0 : unit - p.heads - (kind - 1) * p.kv_heads;
+    const int size = kind == 2 ? p.vdim : p.dim;
+    const int ch0 = kind == 0 ? unit * p.dim : p.heads * p.dim + (kind == 1 ? g * p.dim : p.kv_heads * p.dim + g * p.vdim);
+    const T* in = static_cast<const T*>(p.in) + p.in_off + ch0;
+    const int taps = p.w ? p.taps : 1;
+    float* st = taps > 1 ? p.state + (int64_t)slot * (taps - 1) * p.channels + ch0 : nullptr;
+    const int32_t* trow = kind ? p.table + ((int64_t)slot * p.kv_heads + g) * p.num_tiles : nullptr;
+
+    float wt[TAPS][NP][2], win[TAPS][NP][2], nxt[NP][2];
+#pragma unroll
+    for (int i = 0; i < NP; ++i) {
+        const int d = 2 * lane + 64 * i;
+#pragma unroll
+        for (int b = 0; b < TAPS; ++b) {
+            wt[b][i][0] = wt[b][i][1] = 0.f;
+            win[b][i][0] = win[b][i][1] = 0.f;
+        }
+        nxt[i][0] = nxt[i][1] = 0.f;
+        if (d >= size) continue;
+        const bool second = d + 1 < size;
+        if (p.w) {
+#pragma unroll
+            for (int b = 0; b < TAPS; ++b)
+                if (b < taps) {
+                    wt[b][i][0] = p.w[(int64_t)b * p.channels + ch0 + d];
+                    if (second) wt[b][i][1] = p.w[(int64_t)b * p.channels + ch0 + d + 1];
+                }
+        } else {
+            wt[0][i][0] = wt[0][i][1] = 1.f;
+        }
+        // win[b] = the input b tokens before the CURRENT one; entering the loop it is shifted once
+#pragma unroll
+        for (int b = 0; b + 1 < TAPS; ++b)
+            if (b < taps - 1) {
+                const int t = off - 1 - b;             // offset within the portion
+                if (t >= 0) {
+                    ca_load<T>(in + (int64_t)(row0 - 1 - b) * p.in_stride + d, p.pairs, second, win[b][i][0], win[b][i][1]);
+                } else {
+                    win[b][i][0] = st[(int64_t)(taps - 1 + t) * p.channels + d];
+                    if (second) win[b][i][1] = st[(int64_t)(taps - 1 + t) * p.channels + d + 1];
+                }
+            }
+        ca_load<T>(in + (int64_t)row0 * p.in_stride + d, p.pairs, second, nxt[i][0], nxt[i][1]);
+    }
+
+    for (int t = 0; t < n; ++t) {
+        const int64_t r = row0 + t;
+        float y[NP][2];
+        float ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < NP; ++i) {
+            const int d = 2 * lane + 64 * i;
+#pragma unroll
+            for (int b = TAPS - 1; b > 0; --b) {
+                win[b][i][0] = win[b - 1][i][0];
+                win[b][i][1] = win[b - 1][i][1];
+            }
+            win[0][i][0] = nxt[i][0];
+            win[0][i][1] = nxt[i][1];
+            if (t + 1 < n && d < size)                 // the next token's row is on its way while this one is computed
+                ca_load<T>(in + (r + 1) * p.in_stride + d, p.pairs, d + 1 < size, nxt[i][0], nxt[i][1]);
+            float u = 0.f, v = 0.f;
+#pragma unroll
+            for (int b = 0; b < TAPS; ++b) {
+                u = fmaf(wt[b][i][0], win[b][i][0], u);
+                v = fmaf(wt[b][i][1], win[b][i][1], v);
+            }
+            if (kind < 2 && d < p.rot_dims) {
+                const float2 cs = *reinterpret_cast<const float2*>(p.rope + r * p.rot_dims + d);
+                const float u0 = u;
+                u = u0 * cs.x - v * cs.y;
+                v = v * cs.x + u0 * cs.y;
+            }
+            y[i][0] = u;
+            y[i][1] = v;
+            ss = fmaf(u, u, fmaf(v, v, ss));
+        }
+        if (kind < 2 && p.norm) {
+            const float rn = 1.0f / sqrtf(warp_sum(ss) / (float)size + p.eps);
+#pragma unroll
+            for (int i = 0; i < NP; ++i) { y[i][0] *= rn; y[i][1] *= rn; }
+        }
+        T* dst;
+        if (kind == 0) {
+            dst = static_cast<T*>(p.q_out) + r * p.q_out_stride + ch0;
+        } else {
+            const int pos = pos0 + t;
+            if (pos < 0 || pos / p.tile_size >= p.num_tiles) continue;
+            const int page = trow[pos / p.tile_size];
+            if (page < 0 || page >= p.total_pages) continue;
+            const int64_t prow = (int64_t)page * p.tile_size + pos % p.tile_size;
+            dst = static_cast<T*>(kind == 1 ? p.k_pool : p.v_pool) + prow * size;
+        }
+#pragma unroll
+        for (int i = 0; i < NP; ++i) {
+            const int d = 2 * lane + 64 * i;
+            if (d < size) ca_store<T>(dst + d, p.pairs, d + 1 < size, y[i][0], y[i][1]);
+        }
+    }
+
+    if (off != 0 || taps <= 1) return;
+    // the portion's last taps - 1 raw rows become the state; rows older than the portion move up within the slot
+#pragma unroll
+    for (int i = 0; i < NP; ++i) {
+        const int d = 2 * lane + 64 * i;
+        if (d >= size) continue;
+        const bool second = d + 1 < size;
+        for (int j = 0; j < taps - 1; ++j) {
+            const int t = plen - (taps - 1) + j;
+            float u, v = 0.f;
+            if (t >= 0) {
+                ca_load<T>(in + (int64_t)(row0 + t) * p.in_stride + d, p.pairs, second, u, v);
+            } else {
+                u = st[(int64_t)(taps - 1 + t) * p.channels + d];
+                if (second) v = st[(int64_t)(taps - 1 + t) * p.channels + d + 1];
+            }
+            st[(int64_t)j * p.channels + d] = u;
+            if (second) st[(int64_t)j * p.channels + d + 1] = v;
+        }
+    }
+}
+
+template <typename T, int NP>
+static int ca_launch(const ConvAppendParams& p, cudaStream_t st) {
+    const int units = p.heads + (p.k_pool ? 2 * p.kv_heads : 0);
+    const unsigned grid = (unsigned)(((int64_t)p.num_items * units * 32 + 255) / 256);
+    const int taps = p.w ? p.taps : 1;
+    if (taps <= 1) conv_rope_norm_append_kernel<T, NP, 1><<<grid, 256, 0, st>>>(p);
+    else if (taps <= 4) conv_rope_norm_append_kernel<T, NP, 4><<<grid, 256, 0, st>>>(p);
+    else conv_rope_norm_append_kernel<T, NP, kCaMaxTaps><<<grid, 256, 0, st>>>(p);
+    PA_RETURN_LAUNCH_STATUS();
+}
+
+template <typename T>
+static int ca_dispatch(const ConvAppendParams& p, cudaStream_t st) {
+    const int n = p.k_pool && p.vdim > p.dim ? p.vdim : p.dim;
+    if (n <= 64) return ca_launch<T, 1>(p, st);
+    if (n <= 128) return ca_launch<T, 2>(p, st);
+    if (n <= 256) return ca_launch<T, 4>(p, st);
+    if (n <= 512) return ca_launch<T, 8>(p, st);
+    return PA_ERR_UNSUPPORTED;
+}
+
 constexpr int kMaRows = 32;     // (token, head) rows per CTA
 constexpr int kMaWarps = 8;
 constexpr int kMaRpw = kMaRows / kMaWarps;
@@ -1315,6 +1529,32 @@ PA_API int pa_qk_norm_kv_append(void* d_src, int64_t src_stride, int q_off, int 
                                d_k_gain, eps, static_cast<T*>(d_k_pool), static_cast<T*>(d_v_pool), d_key_scale, d_table,
                                num_slots, num_tiles, total_pages, tile_size, d_row_slot, d_row_pos, rows));
     PA_RETURN_LAUNCH_STATUS();
+}
+
+PA_API int pa_conv_rope_norm_append(const void* d_in, int64_t in_stride, int in_off, int heads, int kv_heads, int dim, int vdim,
+                                    int taps, const float* d_weight, float* d_state, int rot_dims, const float* d_rope,
+                                    int norm, float eps, void* d_q_out, int64_t q_out_stride, void* d_k_pool, void* d_v_pool,
+                                    const int32_t* d_table, int num_slots, int num_tiles, int total_pages, int tile_size,
+                                    const int32_t* d_items, int num_items, int item_tokens, int elem, pa_stream_t stream) {
+    PA_CHECK_ARG(d_in && d_q_out && d_items && num_items >= 0 && heads > 0 && kv_heads > 0 && dim > 0 && vdim > 0 && num_slots > 0);
+    PA_CHECK_ARG(rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= dim && (rot_dims == 0 || d_rope) && (norm == 0 || norm == 1));
+    PA_CHECK_ARG(!d_weight || (taps >= 1 && taps <= kCaMaxTaps && (taps == 1 || d_state) && item_tokens >= taps - 1));
+    PA_CHECK_ARG((d_k_pool != nullptr) == (d_v_pool != nullptr) && d_q_out != d_in);
+    PA_CHECK_ARG(!d_k_pool || (d_table && num_tiles > 0 && total_pages > 0 && tile_size > 0));
+    if (num_items == 0) return PA_OK;
+    ConvAppendParams p;
+    p.in = d_in; p.in_stride = in_stride; p.in_off = in_off; p.heads = heads; p.kv_heads = kv_heads; p.dim = dim; p.vdim = vdim;
+    p.channels = heads * dim + (d_k_pool ? kv_heads * (dim + vdim) : 0);
+    p.rot_dims = rot_dims; p.taps = taps; p.w = d_weight; p.state = d_state; p.rope = d_rope; p.norm = norm; p.eps = eps;
+    p.q_out = d_q_out; p.q_out_stride = q_out_stride; p.k_pool = d_k_pool; p.v_pool = d_v_pool; p.table = d_table;
+    p.num_slots = num_slots; p.num_tiles = num_tiles; p.total_pages = total_pages; p.tile_size = tile_size;
+    p.items = d_items; p.num_items = num_items;
+    const uintptr_t two = 2 * (uintptr_t)(elem == 2 ? 2 : 4);
+    p.pairs = dim % 2 == 0 && vdim % 2 == 0 && in_stride % 2 == 0 && in_off % 2 == 0 && q_out_stride % 2 == 0 &&
+              ((uintptr_t)d_in | (uintptr_t)d_q_out | (uintptr_t)d_k_pool | (uintptr_t)d_v_pool) % two == 0;
+    if (elem == 4) return ca_dispatch<float>(p, as_stream(stream));
+    if (elem == 2) return ca_dispatch<bf16_t>(p, as_stream(stream));
+    return PA_ERR_UNSUPPORTED;
 }
 
 PA_API int pa_masked_attention_mma_tile_tokens(int dim, int vdim, int elem) {

@@ -4,6 +4,7 @@
 // (first row, length, state slot); a row by (state slot, position, row of the previous token or -1).
 //
 //   embedding_rows_kernel     x[r] = table[id[r]] as float
+//   embedding_bigram_kernel   x[r] = embed[id[r]] + bigram[pair of (previous token, token)], optionally kept twice
 //   rms_shift_kernel          RMS norm (scalar or per-channel gain) + optional token shift against the previous token's
 //                             normalised row (from the batch, or from the sequence's state slot at a portion's start)
 //   rms_state_store_kernel    state slot <- normalised row of a portion's last token
@@ -21,7 +22,8 @@
 //                             of the new streams
 //   concat_rows_kernel        [x | x0] of two float row sets in the activation type (input of a looped block)
 //   residual_add_norm2_kernel  the parallel wiring with two norms: x += the sublayers' outputs (routed experts by weight,
-//                             identity experts = the feed-forward's own input row), then BOTH operands of the next layer,
+//                             identity experts = the feed-forward's own input row), plus what a looped block's pass starts
+//                             with (a second float row set and one float row), then BOTH operands of the next layer,
 //                             x / rms(x) * gain1 and x / rms(x) * gain2, from one mean square
 //   poly_norm_kernel          a N(z) + b N(z^2) + c N(z^3) + e per row, N = division by the root mean square of the row
 //   logit_softcap_kernel      cap * tanh(scale * z / cap) on float logits
@@ -39,6 +41,58 @@ __global__ void embedding_rows_kernel(const T* __restrict__ table, const int32_t
     const bool ok = id >= 0 && id < vocab;
     const T* src = table + (int64_t)(ok ? id : 0) * width;
     for (int j = threadIdx.x; j < width; j += blockDim.x) out[(int64_t)r * width + j] = ok ? to_f32<T>(src[j]) * scale : 0.f;
+}
+
+// Row of the pair table: (previous * mul_prev + token * mul_cur) mod buckets, or row `buckets` where there is no previous
+// token (prev = -1).  The result is never negative, whatever the signs.
+__device__ __forceinline__ int64_t bigram_row(int prev, int tok, int64_t mul_prev, int64_t mul_cur, int64_t buckets) {
+    if (prev == -1) return buckets;
+    const int64_t m = ((int64_t)prev * mul_prev + (int64_t)tok * mul_cur) % buckets;
+    return m < 0 ? m + buckets : m;
+}
+
+// VEC columns per access (4: float4 / four bfloat16 in one 8-byte word; the host checks the alignment)
+template <typename T, int VEC>
+__device__ __forceinline__ void load_cols(const T* __restrict__ p, float (&f)[VEC]) {
+    if (VEC == 4 && sizeof(T) == 2) {
+        const uint2 v = *reinterpret_cast<const uint2*>(p);
+        f[0] = __uint_as_float(v.x << 16); f[1 % VEC] = __uint_as_float(v.x & 0xffff0000u);
+        f[2 % VEC] = __uint_as_float(v.y << 16); f[3 % VEC] = __uint_as_float(v.y & 0xffff0000u);
+    } else if (VEC == 4) {
+        const float4 v = *reinterpret_cast<const float4*>(p);
+        f[0] = v.x; f[1 % VEC] = v.y; f[2 % VEC] = v.z; f[3 % VEC] = v.w;
+    } else {
+        f[0] = to_f32<T>(p[0]);
+    }
+}
+template <typename T, int VEC>
+__device__ __forceinline__ void store_cols(T* __restrict__ p, const float (&f)[VEC]) {
+    if (VEC == 4 && sizeof(T) == 2) *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(f[0], f[1 % VEC]), pack_bf16x2(f[2 % VEC], f[3 % VEC]));
+    else if (VEC == 4) *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1 % VEC], f[2 % VEC], f[3 % VEC]);
+    else p[0] = from_f32<T>(f[0]);
+}
+
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256) embedding_bigram_kernel(const T* __restrict__ embed, const T* __restrict__ bigram,
+                                                               const int32_t* __restrict__ ids,
+                                                               const int32_t* __restrict__ prev_ids, int width, int vocab,
+                                                               int64_t buckets, int64_t mul_prev, int64_t mul_cur,
+                                                               float scale, float* __restrict__ out,
+                                                               float* __restrict__ copy) {
+    const int64_t r = blockIdx.x;
+    const int id = ids[r];
+    const bool ok = id >= 0 && id < vocab;
+    const T* a = embed + (int64_t)(ok ? id : 0) * width;
+    const T* b = bigram + bigram_row(prev_ids[r], id, mul_prev, mul_cur, buckets) * width;
+    for (int j = threadIdx.x * VEC; j < width; j += blockDim.x * VEC) {
+        float u[VEC], v[VEC];
+        load_cols<T, VEC>(a + j, u);
+        load_cols<T, VEC>(b + j, v);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) u[i] = ok ? fmaf(u[i], scale, v[i]) : 0.f;
+        store_cols<float, VEC>(out + r * width + j, u);
+        if (copy) store_cols<float, VEC>(copy + r * width + j, u);
+    }
 }
 
 __device__ __forceinline__ float row_inv_rms(const float* __restrict__ xr, int width, float eps, float* sm) {
@@ -407,45 +461,86 @@ __global__ void __launch_bounds__(256) residual_add_prenorm_kernel(float* __rest
 }
 
 // One CTA per row.  s = y + y2 (activation type, optional) + sum_k w[r, k] * e_k, where e_k is the float row
-// routed[(r, k)] of a real expert (sel_id < experts) or the row ident[r] itself (an identity expert); x[r] += s; then
+// routed[(r, k)] of a real expert (sel_id < experts) or the row ident[r] itself (an identity expert); x[r] += s; then, at
+// the start of a looped block's pass, x[r] += base[r] and x[r] += step (float rows, each optional); then
 // next1 = x / rms(x) * gain1 and next2 = x / rms(x) * gain2 (each optional) in the activation type.
-template <typename T>
+template <typename T, int VEC>
 __global__ void __launch_bounds__(256) residual_add_norm2_kernel(float* __restrict__ x, int width, const T* __restrict__ y,
                                                                  const T* __restrict__ y2, const float* __restrict__ routed,
                                                                  const float* __restrict__ sel_w,
                                                                  const int32_t* __restrict__ sel_id, int top, int experts,
-                                                                 const T* __restrict__ ident, float eps,
+                                                                 const T* __restrict__ ident,
+                                                                 const float* __restrict__ base,
+                                                                 const float* __restrict__ step, float eps,
                                                                  const float* __restrict__ gain1, T* __restrict__ next1,
                                                                  const float* __restrict__ gain2, T* __restrict__ next2) {
-    extern __shared__ float row[];                    // [width]
+    extern __shared__ __align__(16) float row[];      // [width]
     __shared__ float sm[32];
     const int64_t r = blockIdx.x;
+    const bool adds = y || y2 || routed || base || step;
     float ss = 0.f;
-    for (int j = threadIdx.x; j < width; j += blockDim.x) {
-        float s = 0.f;
-        if (y) s = to_f32<T>(y[r * width + j]);
-        if (y2) s += to_f32<T>(y2[r * width + j]);
+    for (int j = threadIdx.x * VEC; j < width; j += blockDim.x * VEC) {
+        float v[VEC], s[VEC], t[VEC];
+        load_cols<float, VEC>(x + r * width + j, v);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) s[i] = 0.f;
+        if (y) load_cols<T, VEC>(y + r * width + j, s);
+        if (y2) {
+            load_cols<T, VEC>(y2 + r * width + j, t);
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) s[i] += t[i];
+        }
         if (routed) {
-            float e = 0.f;
+            float e[VEC];
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) e[i] = 0.f;
             for (int k = 0; k < top; ++k) {
                 const bool same = sel_id && sel_id[r * top + k] >= experts;
-                const float v = same ? to_f32<T>(ident[r * width + j]) : routed[(r * top + k) * width + j];
-                e = fmaf(sel_w ? sel_w[r * top + k] : 1.0f, v, e);
+                if (same) load_cols<T, VEC>(ident + r * width + j, t);
+                else load_cols<float, VEC>(routed + (r * top + k) * width + j, t);
+                const float w = sel_w ? sel_w[r * top + k] : 1.0f;
+#pragma unroll
+                for (int i = 0; i < VEC; ++i) e[i] = fmaf(w, t[i], e[i]);
             }
-            s += e;
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) s[i] += e[i];
         }
-        const float v = x[r * width + j] + s;
-        x[r * width + j] = v;
-        row[j] = v;
-        ss = fmaf(v, v, ss);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) v[i] += s[i];
+        if (base) {
+            load_cols<float, VEC>(base + r * width + j, t);
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) v[i] += t[i];
+        }
+        if (step) {
+            load_cols<float, VEC>(step + j, t);
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) v[i] += t[i];
+        }
+        if (adds) store_cols<float, VEC>(x + r * width + j, v);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) {
+            row[j + i] = v[i];
+            ss = fmaf(v[i], v[i], ss);
+        }
     }
     if (!next1 && !next2) return;
     ss = block_sum(ss, sm);
     const float rn = 1.0f / sqrtf(ss / (float)width + eps);
-    for (int j = threadIdx.x; j < width; j += blockDim.x) {
-        const float v = row[j] * rn;
-        if (next1) next1[r * width + j] = from_f32<T>(v * gain1[j]);
-        if (next2) next2[r * width + j] = from_f32<T>(v * gain2[j]);
+    for (int j = threadIdx.x * VEC; j < width; j += blockDim.x * VEC) {     // a thread reads back its own columns
+        float g[VEC], f[VEC];
+        if (next1) {
+            load_cols<float, VEC>(gain1 + j, g);
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) f[i] = row[j + i] * rn * g[i];
+            store_cols<T, VEC>(next1 + r * width + j, f);
+        }
+        if (next2) {
+            load_cols<float, VEC>(gain2 + j, g);
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) f[i] = row[j + i] * rn * g[i];
+            store_cols<T, VEC>(next2 + r * width + j, f);
+        }
     }
 }
 
@@ -617,6 +712,23 @@ PA_API int pa_embedding_rows_scaled(const void* d_table, int elem, const int32_t
     PA_RETURN_LAUNCH_STATUS();
 }
 
+PA_API int pa_embedding_bigram(const void* d_embed, const void* d_bigram, int elem, const int32_t* d_ids,
+                               const int32_t* d_prev_ids, int rows, int width, int vocab, int64_t buckets, int64_t mul_prev,
+                               int64_t mul_cur, float scale, float* d_out, float* d_copy, pa_stream_t stream) {
+    PA_CHECK_ARG(d_embed && d_bigram && d_ids && d_prev_ids && d_out && rows >= 0 && width > 0 && vocab > 0 && buckets > 0);
+    if (rows == 0) return PA_OK;
+    auto al = [](const void* p, int n) { return (uintptr_t)p % n == 0; };
+    const int an = elem == 2 ? 8 : 16;
+    const bool vec = width % 4 == 0 && al(d_embed, an) && al(d_bigram, an) && al(d_out, 16) && al(d_copy, 16);
+#define PA_BIGRAM(VEC)                                                                                              \
+    PA_DISPATCH_ELEM(elem, embedding_bigram_kernel<T, VEC><<<(unsigned)rows, 256, 0, as_stream(stream)>>>(          \
+                               static_cast<const T*>(d_embed), static_cast<const T*>(d_bigram), d_ids, d_prev_ids,  \
+                               width, vocab, buckets, mul_prev, mul_cur, scale, d_out, d_copy))
+    if (vec) { PA_BIGRAM(4); } else { PA_BIGRAM(1); }
+#undef PA_BIGRAM
+    PA_RETURN_LAUNCH_STATUS();
+}
+
 PA_API int pa_embedding_rows(const void* d_table, int elem, const int32_t* d_ids, int rows, int width, int vocab,
                              float* d_out, pa_stream_t stream) {
     return pa_embedding_rows_scaled(d_table, elem, d_ids, rows, width, vocab, 1.0f, d_out, stream);
@@ -756,15 +868,31 @@ PA_API int pa_residual_add_norm2(float* d_x, int64_t rows, int width, const void
                                  const float* d_routed, const float* d_sel_w, const int32_t* d_sel_id, int top,
                                  int experts, const void* d_ident, float eps, const float* d_gain1, void* d_next1,
                                  const float* d_gain2, void* d_next2, int elem, pa_stream_t stream) {
+    return pa_residual_add_norm2_pass(d_x, rows, width, d_y, d_y2, d_routed, d_sel_w, d_sel_id, top, experts, d_ident, nullptr,
+                                      nullptr, eps, d_gain1, d_next1, d_gain2, d_next2, elem, stream);
+}
+
+PA_API int pa_residual_add_norm2_pass(float* d_x, int64_t rows, int width, const void* d_y, const void* d_y2,
+                                      const float* d_routed, const float* d_sel_w, const int32_t* d_sel_id, int top,
+                                      int experts, const void* d_ident, const float* d_base, const float* d_step, float eps,
+                                      const float* d_gain1, void* d_next1, const float* d_gain2, void* d_next2, int elem,
+                                      pa_stream_t stream) {
     PA_CHECK_ARG(d_x && rows >= 0 && width > 0 && (!d_routed || top > 0) && (!d_next1 || d_gain1) && (!d_next2 || d_gain2));
     PA_CHECK_ARG(!d_sel_id || (d_routed && d_ident && experts >= 0));
     if (rows == 0) return PA_OK;
     const size_t smem = (size_t)width * sizeof(float);
     if (smem > 48 * 1024) return PA_ERR_UNSUPPORTED;
-    PA_DISPATCH_ELEM(elem, residual_add_norm2_kernel<T><<<(unsigned)rows, 256, smem, as_stream(stream)>>>(
-                               d_x, width, static_cast<const T*>(d_y), static_cast<const T*>(d_y2), d_routed, d_sel_w,
-                               d_sel_id, top, experts, static_cast<const T*>(d_ident), eps, d_gain1,
-                               static_cast<T*>(d_next1), d_gain2, static_cast<T*>(d_next2)));
+    auto al = [](const void* p, int n) { return (uintptr_t)p % n == 0; };
+    const int an = elem == 2 ? 8 : 16;
+    const bool vec = width % 4 == 0 && al(d_x, 16) && al(d_routed, 16) && al(d_base, 16) && al(d_step, 16) && al(d_gain1, 16) &&
+                     al(d_gain2, 16) && al(d_y, an) && al(d_y2, an) && al(d_ident, an) && al(d_next1, an) && al(d_next2, an);
+#define PA_NORM2(VEC)                                                                                                  \
+    PA_DISPATCH_ELEM(elem, residual_add_norm2_kernel<T, VEC><<<(unsigned)rows, 256, smem, as_stream(stream)>>>(        \
+                               d_x, width, static_cast<const T*>(d_y), static_cast<const T*>(d_y2), d_routed, d_sel_w, \
+                               d_sel_id, top, experts, static_cast<const T*>(d_ident), d_base, d_step, eps, d_gain1,   \
+                               static_cast<T*>(d_next1), d_gain2, static_cast<T*>(d_next2)))
+    if (vec) { PA_NORM2(4); } else { PA_NORM2(1); }
+#undef PA_NORM2
     PA_RETURN_LAUNCH_STATUS();
 }
 

@@ -17,7 +17,7 @@ ACT = {"": 0, None: 0, "none": 0, "relu": 1, "gelu": 2}
 
 _lib = None
 
-_vp, _i32, _i64, _f32, _sz = C.c_void_p, C.c_int, C.c_int64, C.c_float, C.c_size_t
+_vp, _i32, _i64, _f32, _f64, _sz = C.c_void_p, C.c_int, C.c_int64, C.c_float, C.c_double, C.c_size_t
 
 _DECODE_COMMON = [_vp, _i32, _i32, _i32, _i32, _vp, _vp, _i32, _i32, _i32, _i32, _f32, _vp]
 
@@ -185,6 +185,18 @@ _SIGS = {
     "pa_latent_norm_append": ([_vp, _vp, _i32, _i32, _i32, _i32, _i32, _i32, _i32, _i32, _vp, _i64, _i32, _vp, _f32, _vp, _i32,
                                _i32, _vp, _vp, _i64, _vp, _vp, _i32, _i32, _vp], _i32),
     "pa_streams_add_norm": ([_vp, _i32, _vp, _i64, _i32, _i32, _vp, _vp, _vp, _vp, _f32, _vp, _vp, _vp, _vp, _i32, _vp], _i32),
+    # token-pair embedding, block passes that add, convolved + turned + normed projections, sinks on the latent
+    "pa_embedding_bigram": ([_vp, _vp, _i32, _vp, _vp, _i32, _i32, _i32, _i64, _i64, _i64, _f32, _vp, _vp, _vp], _i32),
+    "pa_residual_add_norm2_pass": ([_vp, _i64, _i32, _vp, _vp, _vp, _vp, _vp, _i32, _i32, _vp, _vp, _vp, _f32, _vp, _vp, _vp,
+                                    _vp, _i32, _vp], _i32),
+    "pa_rope_table_scaled": ([_vp, _i32, _i32, _vp, _f64, _vp, _vp], _i32),
+    "pa_latent_turn_append": ([_vp, _vp, _i32, _i32, _i32, _i32, _i32, _i32, _i32, _i32, _vp, _i64, _i32, _vp, _f32, _vp, _vp,
+                               _i64, _i32, _i32, _i32, _vp, _vp, _i32, _i32, _vp], _i32),
+    "pa_gate_rows": ([_vp, _i64, _vp, _i64, _i32, _i64, _vp, _i64, _i32, _vp], _i32),
+    "pa_latent_attention_sink": ([_vp, _i64, _i64, _vp, _i64, _i64, _vp, _vp, _i32, _i32, _i32, _i32, _vp, _i32, _i32, _i32,
+                                  _i32, _f32, _vp, _vp, _i64, _i64, _i32, _i32, _i32, _vp, _sz, _vp], _i32),
+    "pa_conv_rope_norm_append": ([_vp, _i64, _i32, _i32, _i32, _i32, _i32, _i32, _vp, _vp, _i32, _vp, _i32, _f32, _vp, _i64, _vp,
+                                  _vp, _vp, _i32, _i32, _i32, _i32, _vp, _i32, _i32, _i32, _vp], _i32),
     "pa_causal_conv": ([_vp, _i64, _i32, _i32, _i32, _vp, _vp, _i32, _vp, _vp, _i32, _vp, _i64, _i32, _vp], _i32),
 }
 

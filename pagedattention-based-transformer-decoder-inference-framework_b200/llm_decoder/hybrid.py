@@ -1,7 +1,7 @@
 """HybridDecoder -- a config-driven decoder stack over a ragged batch: every layer is one MIXER (picked by the layer's
 `type` from MIXERS) plus an optional FEED-FORWARD (picked by `mlp.kind` from FEED_FORWARDS); the residual stream is
 float.  A DESIGN (config "architecture", table DESIGNS) fixes how a layer is wired and with which constants the
-mechanisms are built.  Four designs are served.
+mechanisms are built.
 
 `Megusun` (wiring 'parallel': mixer and feed-forward both read the same pre-norm output):
 
@@ -66,6 +66,22 @@ mechanisms are built.  Four designs are served.
   ff 'moe'           softmax router over experts + identity outputs, the `top` largest of score + correction, weights = the
                      chosen scores over their sum, on the OUTPUT of silu-gated experts; an identity output returns h itself
 
+`Namudra` (wiring 'streams': the residual as several mixed rows per token, see _stream_layers; windowed sigmoid attention on
+  keys that are the values, latent attention with a half-pair rotation, rotated linear attention with a constant decay).
+
+`Tiradra` (wiring 'parallel_two_norms' with gains stored around zero, N(x; w) = x / sqrt(mean(x^2) + eps) * (1 + w)):
+
+    x0     = embed[token] + bigram[(previous token * a + token * b) mod buckets]   (the table's last row for the first token)
+    pass t of the looped block starts with x += x0 (t > 0), x += step_t            (float, right before its first layer)
+    logits = cap * tanh(head . N(x; w_final) / cap)
+
+  mixer 'attention'  causal softmax attention with grouped key/value heads; biased q, k and v projections pass a short causal
+                     convolution, q and k are rotated (interleaved pairs, frequencies stretched by rot.scaling) and then
+                     divided by their root mean square over the head
+  mixer 'latent_attention'   as in `Domilix` with queries straight from the layer's input, a sink logit per head in the softmax
+                     denominator, and the heads' outputs gated element by element by sigmoid(W_g h)
+  ff 'dense'         W_down (gelu_tanh(W_gate h) * (W_up h))
+
 Every size and constant comes from config.json (or a tensor's shape); the constants a design fixes are the arguments
 the mechanisms are constructed with.  Two precisions: 'bfloat16' (matrix products and their activations in bfloat16
 with float accumulation; norms, shift, recurrence, softmax, routers and the residual in float) and 'float32'
@@ -108,17 +124,54 @@ class _Ctx:
     def empty(self, *shape, dtype=None):
         return torch.empty(shape, dtype=dtype or self.dt, device=self.dev)
 
-    def rope_table(self, dims, base):
-        """[rows][dims / 2][cos, sin] of this step's rows (float), computed once per step and rotation."""
-        key = (dims, base)
+    def rope_table(self, dims, base, scaling=None):
+        """[rows][dims / 2][cos, sin] of this step's rows (float), computed once per step and rotation.  scaling: a
+        stretched rotation (see rotation_scaling), whose factor on cos and sin is part of the table."""
+        key = (dims, base, scaling)
         if key not in self._rope:
             t = None
             if dims > 0:
                 t = self.empty(self.R, dims // 2, 2, dtype=torch.float32)
+            if dims > 0 and scaling is not None:
+                freqs, mult = self.model.rotation_freqs(dims, base, scaling)
+                _chk(self.lib.pa_rope_table_scaled(self.batch.row_pos.data_ptr(), self.R, dims, freqs.data_ptr(), mult,
+                                                   t.data_ptr(), _cabi.stream()), "pa_rope_table_scaled")
+            elif dims > 0:
                 _chk(self.lib.pa_rope_table(self.batch.row_pos.data_ptr(), self.R, dims, base, t.data_ptr(), _cabi.stream()),
                      "pa_rope_table")
             self._rope[key] = t
         return self._rope[key]
+
+
+# -------------------------------------------------------------------------------------------------------------- rotation
+def rotation_scaling(rot):
+    """cfg rot.scaling {factor, original, fast, slow} as a hashable tuple (None: a plain rotation)."""
+    sc = (rot or {}).get("scaling")
+    if not sc:
+        return None
+    out = tuple(float(sc[k]) for k in ("factor", "original", "fast", "slow"))
+    if min(out) <= 0.0:
+        raise ValueError("rot.scaling: factor, original, fast and slow must be positive")
+    return out
+
+
+def scaled_frequencies(dims, base, scaling):
+    """Angle per position of every pair of a rotation whose slow pairs are stretched (YaRN: Peng et al., "YaRN: Efficient
+    Context Window Extension of Large Language Models"), and the factor on cos and sin.  A pair that turns more than
+    `fast` times over `original` positions keeps base^(-2i / dims), one that turns less than `slow` times is divided by
+    `factor`, and in between the two are blended linearly over the pair index."""
+    factor, original, fast, slow = scaling
+
+    def pair_of(turns):
+        return dims * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
+
+    lo, hi = max(math.floor(pair_of(fast)), 0), min(math.ceil(pair_of(slow)), dims - 1)
+    freqs = []
+    for i in range(dims // 2):
+        f = base ** (-2.0 * i / dims)
+        ramp = min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0)
+        freqs.append(f / factor * ramp + f * (1.0 - ramp))
+    return freqs, 0.1 * math.log(factor) + 1.0
 
 
 # ---------------------------------------------------------------------------------------------------------------- mixers
@@ -229,16 +282,25 @@ class LatentAttentionMixer:
     """Attention through a low-rank latent over a paged pool with ONE row per token (KVTileCache with one key/value head
     and no value pool: row = [c | kr]).  The per-head key and value maps are applied on the query side and after the
     weighted sum (pa_head_linear), so a step reads kv_rank + rot_dim values per cached token whatever the head count.
-    A design picks the pairs of the rotation (pairing 'neighbours': (2i, 2i + 1), or 'halves': (i, i + dims / 2)) and
-    whether every head's output is gated by sigmoid(W_g h) (head_gate)."""
+    A design picks
+
+      pairing      the pairs of the rotation: 'neighbours' (2i, 2i + 1), or 'halves' (i, i + dims / 2)
+      q_latent     whether the queries pass a normed latent of cfg q_rank ('<prefix>dq', 'dq.norm', 'uq') or come straight
+                   from the layer's input ('<prefix>q')
+      gate         'head': every head's output times its number of sigmoid(W_g h); 'elements': every element of the heads'
+                   outputs times its own; None
+      sink         a learned logit per head ('<prefix>sink') in the softmax denominator, without key or value, unscaled"""
     kind = "latent_attention"
 
-    def __init__(self, model, prefix, cfg, W, pairing="neighbours", head_gate=True):
-        self.pairing, self.head_gate = ROPE_PAIRING[pairing], bool(head_gate)
+    def __init__(self, model, prefix, cfg, W, pairing="neighbours", q_latent=True, gate="head", sink=False):
+        if gate not in ("head", "elements", None):
+            raise ValueError(f"unknown gate {gate!r}")
+        self.pairing, self.gate, self.q_latent = ROPE_PAIRING[pairing], gate, bool(q_latent)
         H, self.dim, self.rot_dim, self.vdim = int(cfg["heads"]), int(cfg["dim"]), int(cfg["rot_dim"]), int(cfg["vdim"])
-        self.heads, self.kv_rank, self.q_rank = H, int(cfg["kv_rank"]), int(cfg["q_rank"])
+        self.heads, self.kv_rank, self.q_rank = H, int(cfg["kv_rank"]), int(cfg["q_rank"]) if self.q_latent else 0
         rot = cfg.get("rot") or {}
         self.rot_dims, self.rot_base = int(rot.get("dims", self.rot_dim)), float(rot.get("base", 10000.0))
+        self.rot_scaling = rotation_scaling(rot)
         if self.rot_dims > self.rot_dim or self.rot_dims % 2:
             raise ValueError("rot.dims must be even and at most rot_dim")
         self.scale = float(cfg["scale"])
@@ -246,18 +308,25 @@ class LatentAttentionMixer:
         self.own_kv = self.kv_from is None
         qd, kd = self.dim + self.rot_dim, self.kv_rank + self.rot_dim
         self.qd, self.kd = qd, kd
-        for name, shape in (("dq", (self.q_rank, model.width)), ("uq", (H * qd, self.q_rank)), ("uk", (H * self.dim, self.kv_rank)),
-                            ("uv", (H * self.vdim, self.kv_rank)), ("o", (model.width, H * self.vdim))) + (
-                                (("g", (H, model.width)),) if self.head_gate else ()):
+        gate_cols = {"head": H, "elements": H * self.vdim, None: 0}[gate]
+        shapes = [("uk", (H * self.dim, self.kv_rank)), ("uv", (H * self.vdim, self.kv_rank)), ("o", (model.width, H * self.vdim))]
+        shapes += ([("dq", (self.q_rank, model.width)), ("uq", (H * qd, self.q_rank))] if self.q_latent else
+                   [("q", (H * qd, model.width))])
+        shapes += [("g", (gate_cols, model.width))] if gate else []
+        shapes += [("sink", (H,))] if sink else []
+        for name, shape in shapes:
             if tuple(W[prefix + name].shape) != shape:
                 raise ValueError(f"{prefix}{name}: shape {tuple(W[prefix + name].shape)} does not match the config {shape}")
-        # one product for everything that reads the layer's input: [dq | dkv (own pool only) | g (gated only)]
-        parts = ([W[prefix + "dq"]] + ([W[prefix + "dkv"]] if self.own_kv else []) + ([W[prefix + "g"]] if self.head_gate else []))
+        # one product for everything that reads the layer's input: [dq or q | dkv (own pool only) | g (gated only)]
+        parts = ([W[prefix + ("dq" if self.q_latent else "q")]] + ([W[prefix + "dkv"]] if self.own_kv else []) +
+                 ([W[prefix + "g"]] if gate else []))
         self.w_in = model._weight(torch.cat(parts, 0))
-        self.c_off = self.q_rank
-        self.g_off = self.q_rank + (kd if self.own_kv else 0)
-        self.dq_gain = model._f32(W[prefix + "dq.norm"])
-        self.w_uq = model._weight(W[prefix + "uq"])
+        self.c_off = int(parts[0].shape[0])
+        self.g_off = self.c_off + (kd if self.own_kv else 0)
+        self.sink = model._f32(W[prefix + "sink"]) if sink else None
+        if self.q_latent:
+            self.dq_gain = model._f32(W[prefix + "dq.norm"])
+            self.w_uq = model._weight(W[prefix + "uq"])
         self.w_uk = model._weight_raw(W[prefix + "uk"].reshape(H, self.dim, self.kv_rank))                    # [H][dim][kv_rank]
         self.w_uv = model._weight_raw(W[prefix + "uv"].reshape(H, self.vdim, self.kv_rank).transpose(1, 2))   # [H][kv_rank][vdim]
         self.w_o = model._weight(W[prefix + "o"])
@@ -271,8 +340,8 @@ class LatentAttentionMixer:
             src = model.layers[j].mixer if 0 <= j < len(model.layers) else None
             if not isinstance(src, LatentAttentionMixer) or not src.own_kv:
                 raise ValueError(f"{prefix}: kv_from must name an earlier latent-attention layer with a pool of its own")
-            if (src.kv_rank, src.rot_dim, src.rot_dims, src.rot_base, src.pairing) != (self.kv_rank, self.rot_dim, self.rot_dims,
-                                                                                       self.rot_base, self.pairing):
+            same = ("kv_rank", "rot_dim", "rot_dims", "rot_base", "rot_scaling", "pairing")
+            if any(getattr(src, n) != getattr(self, n) for n in same):
                 raise ValueError(f"{prefix}: kv_rank, rot_dim and rotation must equal those of layer {j}")
             self.kv = src.kv
         self.tile_tokens = model._lib.pa_latent_attention_tile_tokens(H)
@@ -320,38 +389,53 @@ class LatentAttentionMixer:
             nsplit = latent_key_splits(ntiles * math.ceil(H / rows_per_cta), longest, c.model.sm_count)
             if nsplit > 1:
                 ws = c.empty(lib.pa_latent_attention_workspace_bytes(ntiles, H, kvr, nsplit), dtype=torch.uint8)
-            st = lib.pa_latent_attention(ql.data_ptr(), kvr, R * kvr, q.data_ptr() + self.dim * c.elem, q.stride(0), self.qd,
-                                         kv.key_buffer_.data_ptr(), table.data_ptr(), pt.num_beams_, pt.num_tiles_,
-                                         kv.total_pages_, kv.tile_size_, tiles.data_ptr(), ntiles, H, kvr, self.rot_dim,
-                                         self.scale, lat.data_ptr(), kvr, R * kvr, c.elem, nsplit,
-                                         (3 if kind == 1 else 2) if mma else 0, _cabi.ptr(ws),
-                                         ws.numel() if ws is not None else 0, s)
+            st = lib.pa_latent_attention_sink(ql.data_ptr(), kvr, R * kvr, q.data_ptr() + self.dim * c.elem, q.stride(0), self.qd,
+                                              kv.key_buffer_.data_ptr(), table.data_ptr(), pt.num_beams_, pt.num_tiles_,
+                                              kv.total_pages_, kv.tile_size_, tiles.data_ptr(), ntiles, H, kvr, self.rot_dim,
+                                              self.scale, _cabi.ptr(self.sink), lat.data_ptr(), kvr, R * kvr, c.elem, nsplit,
+                                              (3 if kind == 1 else 2) if mma else 0, _cabi.ptr(ws),
+                                              ws.numel() if ws is not None else 0, s)
             if mma and st == _cabi.PA_ERR_UNSUPPORTED:
                 return False
-            _chk(st, "pa_latent_attention")
+            _chk(st, "pa_latent_attention_sink")
         return True
 
-    def forward(self, c, h):
+    def _queries(self, c, proj):
+        """The queries of this step's rows ([R, heads * (dim + rot_dim)] with any row stride), rotated; the new pool rows of
+        a layer with a pool of its own go out in the same launch as the norm of the query latent, or, without one, as the
+        rotation of the queries (in place, in proj)."""
         b, lib, kv, s, R, H = c.batch, c.lib, self.kv, _cabi.stream(), c.R, self.heads
-        proj = c.model._linear(h, self.w_in)
-        cq = c.empty(R, self.q_rank)
-        rope = c.rope_table(self.rot_dims, self.rot_base)
+        rope = c.rope_table(self.rot_dims, self.rot_base, self.rot_scaling)
         pt = kv.page_table_
         table = pt.device_data()
-        if self.own_kv:     # the norm of the query latent and the new pool rows: one launch
-            _chk(lib.pa_latent_norm_append(kv.key_buffer_.data_ptr(), table.data_ptr(), pt.num_beams_, pt.num_tiles_,
-                                           kv.total_pages_, kv.tile_size_, self.kv_rank, self.rot_dim, self.rot_dims,
-                                           self.pairing, proj.data_ptr(), proj.stride(0), self.c_off,
-                                           self.dkv_gain.data_ptr(), c.model.eps, _cabi.ptr(rope), 0, self.q_rank,
-                                           self.dq_gain.data_ptr(), cq.data_ptr(), self.q_rank, b.row_slot.data_ptr(),
-                                           b.row_pos.data_ptr(), R, c.elem, s), "pa_latent_norm_append")
-        else:
-            _chk(lib.pa_rms_norm_rows(proj.data_ptr(), proj.stride(0), 0, self.q_rank, c.model.eps, self.dq_gain.data_ptr(),
-                                      cq.data_ptr(), self.q_rank, R, c.elem, s), "pa_rms_norm_rows")
-        q = c.model._linear(cq, self.w_uq)
+        pool = (kv.key_buffer_.data_ptr(), table.data_ptr(), pt.num_beams_, pt.num_tiles_, kv.total_pages_, kv.tile_size_,
+                self.kv_rank, self.rot_dim, self.rot_dims, self.pairing)
+        if self.own_kv:
+            src = (proj.data_ptr(), proj.stride(0), self.c_off, self.dkv_gain.data_ptr(), c.model.eps, _cabi.ptr(rope))
+        rows = (b.row_slot.data_ptr(), b.row_pos.data_ptr(), R, c.elem, s)
+        if self.own_kv and not self.q_latent:
+            _chk(lib.pa_latent_turn_append(*pool, *src, proj.data_ptr(), proj.stride(0), self.dim, H, self.qd, *rows),
+                 "pa_latent_turn_append")
+            return proj
+        q = proj
+        if self.q_latent:
+            cq = c.empty(R, self.q_rank)
+            if self.own_kv:
+                _chk(lib.pa_latent_norm_append(*pool, *src, 0, self.q_rank, self.dq_gain.data_ptr(), cq.data_ptr(), self.q_rank,
+                                               *rows), "pa_latent_norm_append")
+            else:
+                _chk(lib.pa_rms_norm_rows(proj.data_ptr(), proj.stride(0), 0, self.q_rank, c.model.eps, self.dq_gain.data_ptr(),
+                                          cq.data_ptr(), self.q_rank, R, c.elem, s), "pa_rms_norm_rows")
+            q = c.model._linear(cq, self.w_uq)
         if self.rot_dims:
             _chk(lib.pa_rope_rows_paired(q.data_ptr(), q.stride(0), self.dim, self.qd, H, self.rot_dims, _cabi.ptr(rope),
                                          self.pairing, R, c.elem, s), "pa_rope_rows_paired")
+        return q
+
+    def forward(self, c, h):
+        lib, s, R, H = c.lib, _cabi.stream(), c.R, self.heads
+        proj = c.model._linear(h, self.w_in)
+        q = self._queries(c, proj)
         kvr = self.kv_rank
         ql = self._head_linear(c, q, q.stride(0), self.qd, self.w_uk, self.dim, kvr)          # [H, R, kv_rank]
         lat = c.empty(H, R, kvr)
@@ -359,9 +443,12 @@ class LatentAttentionMixer:
             self.mma_tokens = 0         # a stride or an alignment the tensor-core kernel does not take: the float kernel
         if self.mma_tokens == 0:
             self._attend(c, q, ql, lat, False)
-        if not self.head_gate:
-            ov = self._head_linear(c, lat, kvr, R * kvr, self.w_uv, kvr, self.vdim, by_row=True)
-            return c.model._linear(ov.view(R, H * self.vdim), self.w_o)
+        if self.gate != "head":
+            ov = self._head_linear(c, lat, kvr, R * kvr, self.w_uv, kvr, self.vdim, by_row=True).view(R, H * self.vdim)
+            if self.gate == "elements":
+                _chk(lib.pa_gate_rows(ov.data_ptr(), ov.stride(0), proj.data_ptr() + self.g_off * c.elem, proj.stride(0),
+                                      H * self.vdim, R, ov.data_ptr(), ov.stride(0), c.elem, s), "pa_gate_rows")
+            return c.model._linear(ov, self.w_o)
         ov = self._head_linear(c, lat, kvr, R * kvr, self.w_uv, kvr, self.vdim)               # [H, R, vdim]
         og = c.empty(R, H * self.vdim)
         _chk(lib.pa_head_gate(ov.data_ptr(), self.vdim, R * self.vdim, proj.data_ptr() + self.g_off * c.elem, proj.stride(0),
@@ -371,6 +458,7 @@ class LatentAttentionMixer:
 
 MASK_KIND = {"causal": 0, "window": 1, "chunk": 2}
 CONV_CHUNK = 64           # tokens per work item of the causal convolution
+APPEND_CHUNK = 16         # tokens per work item of the fused convolution + rotation + norm + append
 DECAY_CHUNK = 64          # tokens per chunk of the chunked matrix-state scan
 DECAY_CHUNKED_FROM = 256  # portions at least this long use it
 
@@ -390,16 +478,18 @@ class MaskedAttention:
     a learned table '<prefix>rel' [buckets, heads] over log_distance_bucket(distance, buckets, cfg bias_max)), whether cfg
     'softcap' caps the scores, and
 
-      proj_bias    whether the four projections have biases ('<name>.b')
+      proj_bias    whether the four projections have biases ('<name>.b'); 'qkv': all but the output product
       conv         a short causal convolution (cfg 'conv' taps, weights '<name>.conv' [channels, taps], no bias, no
                    activation) on q, k and v right after the projection; the last taps - 1 projected rows are state
-      rot          interleaved-pair rotation of the first cfg rot.dims dimensions of every q and k head (cfg rot.base)
+      rot          interleaved-pair rotation of the first cfg rot.dims dimensions of every q and k head (cfg rot.base; cfg
+                   rot.scaling stretches its slow pairs, see scaled_frequencies)
       rot_values   values cached turned by their own position over all of vdim (same pairs, angles p * base^(-2m / vdim));
                    every head's output is turned back by the query's position inside the attention kernels
       head_temp    a learned factor per query head on the scaled dot products ('<prefix>temp')
       sink         'learned': a logit per head ('<prefix>sink') in the softmax denominator, without key or value;
                    'zero': the same with logit 0 (one added to the denominator)
-      qk_norm      every query and key head divided by its root mean square, times '<prefix>q.norm' / '<prefix>k.norm' [dim]
+      qk_norm      every query and key head divided by its root mean square, times '<prefix>q.norm' / '<prefix>k.norm' [dim];
+                   'turned': divided after the rotation, without a gain
       values       'own', or 'keys': there is no value projection, the values are the keys before their norm -- the pool
                    holds ONE row per key (as projected) and its inverse root mean square beside it; the norm's gain goes
                    to the query side
@@ -427,7 +517,8 @@ class MaskedAttention:
         self.kv_from = cfg.get("kv_from")
         self.own_kv = self.kv_from is None
         H = self.heads
-        self.qk_norm, self.keys_as_values = bool(qk_norm), values == "keys"
+        self.turned_norm = qk_norm == "turned"
+        self.qk_norm, self.keys_as_values = bool(qk_norm) and not self.turned_norm, values == "keys"
         if values not in ("own", "keys") or weights not in ("softmax", "sigmoid"):
             raise ValueError(f"unknown values {values!r} or weights {weights!r}")
         self.sigmoid = 1 if weights == "sigmoid" else 0
@@ -435,6 +526,8 @@ class MaskedAttention:
             raise ValueError(f"{prefix}: values that are the keys need vdim = dim and the query / key norm")
         if self.qk_norm and (rot or rot_values or not self.own_kv):
             raise ValueError(f"{prefix}: the query / key norm is served without rotation and on a pool of the layer's own")
+        if self.turned_norm and (rot_values or not self.own_kv):
+            raise ValueError(f"{prefix}: the norm after the rotation is served without turned values, on a pool of the layer's own")
         if self.sigmoid and sink is not None:
             raise ValueError(f"{prefix}: sigmoid weights have no denominator for a sink")
         shapes = (("q", H * self.dim),)
@@ -468,7 +561,7 @@ class MaskedAttention:
             if tuple(W[prefix + "pb"].shape) != (H,):
                 raise ValueError(f"{prefix}pb: one number per head expected")
             self.head_bias = model._f32(W[prefix + "pb"])
-        self.w_o, self.b_o = model._weight(W[prefix + "o"]), model._bias(W[prefix + "o.b"]) if proj_bias else None
+        self.w_o, self.b_o = model._weight(W[prefix + "o"]), model._bias(W[prefix + "o.b"]) if proj_bias is True else None
         self.taps, self.conv_w = 0, None
         if conv:
             self.taps = int(W[prefix + "q.conv"].shape[-1])     # the tensors' shape gives the taps; cfg 'conv' must agree
@@ -480,10 +573,15 @@ class MaskedAttention:
                 if tuple(W[prefix + name + ".conv"].shape) != (rows, self.taps):
                     raise ValueError(f"{prefix}{name}.conv: shape does not match the config")
             self.conv_w = model._f32(torch.cat([W[prefix + n + ".conv"] for n, _ in shapes], 0))
-        self.rot_dims, self.rot_base, self.rot_values = 0, 0.0, bool(rot_values)
+            # [taps][channels], entry b = the weight b tokens back, for the fused launch
+            self.conv_wt = self.conv_w.flip(1).t().contiguous()
+        self.rot_dims, self.rot_base, self.rot_values, self.rot_scaling = 0, 0.0, bool(rot_values), None
         if rot or rot_values:
             self.rot_base = float(cfg["rot"]["base"])
+        if rot_values and rotation_scaling(cfg["rot"]):
+            raise ValueError(f"{prefix}: turned values are served with a plain rotation")
         if rot:
+            self.rot_scaling = rotation_scaling(cfg["rot"])
             self.rot_dims = int(cfg["rot"]["dims"])
             if self.rot_dims % 2 or self.rot_dims > self.dim:
                 raise ValueError(f"{prefix}: rot.dims must be even and at most dim")
@@ -510,8 +608,8 @@ class MaskedAttention:
             src = getattr(src, "core", None)
             if not isinstance(src, MaskedAttention) or not src.own_kv:
                 raise ValueError(f"{prefix}: kv_from must name an earlier attention layer with a pool of its own")
-            mine = (self.kv_heads, self.dim, self.vdim, self.rot_dims, self.rot_base, self.rot_values)
-            if (src.kv_heads, src.dim, src.vdim, src.rot_dims, src.rot_base, src.rot_values) != mine:
+            same = ("kv_heads", "dim", "vdim", "rot_dims", "rot_base", "rot_scaling", "rot_values", "turned_norm")
+            if any(getattr(src, n) != getattr(self, n) for n in same):
                 raise ValueError(f"{prefix}: key/value heads, sizes and rotation must equal those of layer {j}")
             self._src = src
         self.bias_kind, self.bias_len, self.bias = 0, 0, None
@@ -549,6 +647,18 @@ class MaskedAttention:
         """Convolution and rotation of this step's q | k | v rows, then the new keys and values go to the pool.  Returns
         the buffer and column offset the attention kernels read the queries from."""
         b, lib, s, R = c.batch, c.lib, _cabi.stream(), c.R
+        if self.turned_norm:        # convolution, rotation, norm and append: one launch
+            kv, pt = self.kv, self.kv.page_table_
+            items, n = b.portion_items(APPEND_CHUNK)
+            q = c.empty(R, self.q_cols)
+            _chk(lib.pa_conv_rope_norm_append(
+                proj.data_ptr(), proj.stride(0), off, self.heads, self.kv_heads, self.dim, self.vdim, self.taps,
+                _cabi.ptr(self.conv_wt) if self.taps else None, _cabi.ptr(self.conv_state), self.rot_dims,
+                _cabi.ptr(c.rope_table(self.rot_dims, self.rot_base, self.rot_scaling)), 1, c.model.eps, q.data_ptr(), self.q_cols,
+                kv.key_buffer_.data_ptr(), kv.value_buffer_.data_ptr(), pt.device_data().data_ptr(), pt.num_beams_,
+                pt.num_tiles_, kv.total_pages_, kv.tile_size_, items.data_ptr(), n, APPEND_CHUNK, c.elem, s),
+                "pa_conv_rope_norm_append")
+            return q, 0
         if self.taps:
             chunks, nch, _s0, _sn = b.chunk_items(CONV_CHUNK)
             y = c.empty(R, self.qkv_cols)
@@ -566,7 +676,7 @@ class MaskedAttention:
             pt = kv.page_table_
             own = self.own_kv
             _chk(lib.pa_rope_kv_append(proj.data_ptr(), proj.stride(0), off, k_off, v_off, self.heads, self.kv_heads, self.dim,
-                                       self.vdim, self.rot_dims, _cabi.ptr(c.rope_table(self.rot_dims, self.rot_base)),
+                                       self.vdim, self.rot_dims, _cabi.ptr(c.rope_table(self.rot_dims, self.rot_base, self.rot_scaling)),
                                        _cabi.ptr(c.rope_table(self.vdim, self.rot_base)) if self.rot_values else None,
                                        kv.key_buffer_.data_ptr() if own else None,
                                        kv.value_buffer_.data_ptr() if own else None, pt.device_data().data_ptr(),
@@ -971,7 +1081,7 @@ DESIGNS = {
                                             "moe": dict(score="sigmoid", weight_on="input", act="silu", gated=True)}),
     "Domilix": dict(wiring="post_norm", ff={"dense": dict(act="relu", gated=True),
                                             "moe": dict(score="softmax_chosen", weight_on="output", act="relu2", gated=False)}),
-    "Dubarax": dict(wiring="pre_norm", loop_entry=True,
+    "Dubarax": dict(wiring="pre_norm", loop_entry="product",
                     mixers={"attention": (SoftmaxAttentionMixer, dict(mask="window", bias="bucket", softcap=True)),
                             "parallel": (ParallelMixer, dict(left=dict(mask="chunk", bias="slope", slope_exp=8.0))),
                             "mamba2": (Mamba2Mixer, {})},
@@ -988,8 +1098,13 @@ DESIGNS = {
                     mixers={"retention": (LinearAttentionMixer, dict(act=None, rot=True, key_scale=True, norm="head", gate="silu")),
                             "attention": (SoftmaxAttentionMixer, dict(mask="window", proj_bias=False, qk_norm=True, values="keys",
                                                                       weights="sigmoid", head_bias=True, gate=True)),
-                            "latent_attention": (LatentAttentionMixer, dict(pairing="halves", head_gate=False))},
+                            "latent_attention": (LatentAttentionMixer, dict(pairing="halves", gate=None))},
                     ff={"dense": dict(act="silu", gated=True)}),
+    "Tiradra": dict(wiring="parallel_two_norms", gains="around_zero", loop_entry="add",
+                    mixers={"attention": (SoftmaxAttentionMixer, dict(mask="causal", proj_bias="qkv", conv=True, rot=True,
+                                                                      qk_norm="turned")),
+                            "latent_attention": (LatentAttentionMixer, dict(q_latent=False, gate="elements", sink=True))},
+                    ff={"dense": dict(act="gelu_tanh", gated=True)}),
 }
 
 
@@ -1014,19 +1129,27 @@ class HybridDecoder:
         self.mult = float(config.get("residual_mult", 1.0))
         self.embed_scale = float((config.get("embedding") or {}).get("scale", 1.0))
         self.states = SequenceStateCache(max_seqs, max_tokens, tile_size, self.device)
-        self._ws = None
+        self._ws, self._rot_freqs = None, {}
         W = weights
         if tuple(W["embed"].shape) != (self.vocab, self.width):
             raise ValueError("embed does not match config vocab / width")
         self.embed = W["embed"].to(self.device, self.act_dtype).contiguous()
+        self.bigram = None
+        bg = (config.get("embedding") or {}).get("bigram")
+        if bg:      # a second table indexed by (previous token, token); its last row is for a sequence's first token
+            self.bigram_consts = (int(bg["buckets"]), int(bg["mul_prev"]), int(bg["mul_cur"]))
+            if self.bigram_consts[0] < 1 or tuple(W["bigram"].shape) != (self.bigram_consts[0] + 1, self.width):
+                raise ValueError("bigram does not match config embedding.bigram.buckets / width")
+            self.bigram = W["bigram"].to(self.device, self.act_dtype).contiguous()
+            self.states.track_tokens = True
         self.head = self._weight(W["head"])
         self.streams = int(config.get("streams") or 0)
         if self.wiring == "streams" and self.streams == 0:
             self.wiring = "pre_norm"        # a single residual without stream mixing
         post, pre, par2 = self.wiring == "post_norm", self.wiring in ("pre_norm", "streams"), self.wiring == "parallel_two_norms"
         self.final_gain = 1.0 if post or pre or par2 else float(W["final.norm"].to(torch.float32))
-        self.final_gain_vec = (self._f32(W["final.norm"].reshape(-1)) if post or par2 else
-                               self._gain1p(W["final.norm"]) if pre else None)
+        gain = self._gain1p if pre or self.design.get("gains") == "around_zero" else lambda t: self._f32(t.reshape(-1))
+        self.final_gain_vec = gain(W["final.norm"]) if post or par2 or pre else None
         if self.final_gain_vec is not None and self.final_gain_vec.numel() != self.width:
             raise ValueError("final.norm does not match width")
         ls, lc_ = config.get("logit_scale"), config.get("logit_softcap")      # absent or null: no scaling / no cap
@@ -1037,8 +1160,8 @@ class HybridDecoder:
             L = _Layer()
             p = f"l{i}."
             if post or par2:    # per-channel gains: post-norm on the two sublayers' outputs; two norms of the same x in front of them
-                L.gain1 = self._f32(W[p + "norm1"].reshape(-1))
-                L.gain2 = self._f32(W[p + "norm2"].reshape(-1)) if lc.get("mlp") else None
+                L.gain1 = gain(W[p + "norm1"])
+                L.gain2 = gain(W[p + "norm2"]) if lc.get("mlp") else None
                 L.shift = L.prev = None
             elif pre:   # per-channel gains of the norms in front of the two sublayers, stored around zero
                 L.gain1 = self._gain1p(W[p + "norm1"])
@@ -1069,24 +1192,27 @@ class HybridDecoder:
     def _build_runs(self, loop, W):
         """The order in which layers RUN: (layer, mixer, pass number or None).  A looped block [start, stop) runs `times`
         times in a row with the same weights; every pass after the first gets mixers with a cache / state of their own
-        (new_pass).  In a design with `loop_entry` its first run carries the pass number: the block input
-        x <- W_in [x | x0] + step[t] comes first."""
+        (new_pass).  In a design with `loop_entry` its first run carries the pass number, and the block input comes first:
+        'product': x <- W_in [x | x0] + step[t];  'add': x += x0 in every pass but the first, then x += step[t]."""
         n = len(self.layers)
         self.loop_in = self.loop_step = None
         if not loop or int(loop.get("times", 0)) < 1 or int(loop["stop"]) <= int(loop["start"]):
             self.runs = [(L, L.mixer, None) for L in self.layers]
             return
-        if self.wiring not in ("pre_norm", "streams"):
-            raise ValueError("looped blocks are served in the pre-norm and stream wirings")
+        entry = self.design.get("loop_entry")
+        if self.wiring not in ("pre_norm", "streams", "parallel_two_norms") or (self.wiring == "parallel_two_norms" and entry != "add"):
+            raise ValueError("looped blocks are served in the pre-norm and stream wirings, and in the two-norm wiring whose passes add")
         a, b, times = int(loop["start"]), int(loop["stop"]), int(loop["times"])
         if not 0 <= a < b <= n:
             raise ValueError("loop: start / stop outside the layer list")
-        entry = bool(self.design.get("loop_entry"))
         if entry:
-            if tuple(W["loop.in"].shape) != (self.width, 2 * self.width) or tuple(W["loop.step"].shape) != (times, self.width):
-                raise ValueError("loop.in / loop.step do not match width / times")
-            self.loop_in = self._weight(W["loop.in"])
+            if tuple(W["loop.step"].shape) != (times, self.width):
+                raise ValueError("loop.step does not match times / width")
             self.loop_step = self._f32(W["loop.step"])
+        if entry == "product":
+            if tuple(W["loop.in"].shape) != (self.width, 2 * self.width):
+                raise ValueError("loop.in does not match width")
+            self.loop_in = self._weight(W["loop.in"])
         self.runs = [(L, L.mixer, None) for L in self.layers[:a]]
         for t in range(times):
             for i in range(a, b):
@@ -1105,6 +1231,14 @@ class HybridDecoder:
     # ---- weights ----------------------------------------------------------------------------------------------------
     def _f32(self, t):
         return t.to(torch.float32).to(self.device).contiguous()
+
+    def rotation_freqs(self, dims, base, scaling):
+        """(double device tensor of a stretched rotation's frequencies, factor on cos and sin), made once per rotation."""
+        key = (dims, base, scaling)
+        if key not in self._rot_freqs:
+            freqs, mult = scaled_frequencies(dims, base, scaling)
+            self._rot_freqs[key] = (torch.tensor(freqs, dtype=torch.float64, device=self.device), mult)
+        return self._rot_freqs[key]
 
     def _gain1p(self, t):
         """1 + w of a norm weight stored around zero (float)."""
@@ -1158,14 +1292,25 @@ class HybridDecoder:
         c = _Ctx(self, batch)
         lib, R, W, s = self._lib, batch.rows, self.width, _cabi.stream()
         x = torch.empty((R, W), dtype=torch.float32, device=self.device)
-        _chk(lib.pa_embedding_rows_scaled(self.embed.data_ptr(), c.elem, batch.ids.data_ptr(), R, W, self.vocab,
-                                          self.embed_scale, x.data_ptr(), s), "pa_embedding_rows_scaled")
+        x0 = None       # the embedding output, kept where a block's later passes add it again
+        if self.loop_step is not None and self.loop_in is None and self.loop_step.shape[0] > 1:
+            x0 = torch.empty_like(x)
+        if self.bigram is not None:
+            buckets, mul_prev, mul_cur = self.bigram_consts
+            _chk(lib.pa_embedding_bigram(self.embed.data_ptr(), self.bigram.data_ptr(), c.elem, batch.ids.data_ptr(),
+                                         batch.prev_ids.data_ptr(), R, W, self.vocab, buckets, mul_prev, mul_cur,
+                                         self.embed_scale, x.data_ptr(), _cabi.ptr(x0), s), "pa_embedding_bigram")
+        else:
+            _chk(lib.pa_embedding_rows_scaled(self.embed.data_ptr(), c.elem, batch.ids.data_ptr(), R, W, self.vocab,
+                                              self.embed_scale, x.data_ptr(), s), "pa_embedding_rows_scaled")
+            if x0 is not None:
+                x0.copy_(x)
         if self.wiring == "post_norm":
             self._post_norm_layers(c, x)
         elif self.wiring == "pre_norm":
             x = self._pre_norm_layers(c, x)
         elif self.wiring == "parallel_two_norms":
-            self._parallel_two_norm_layers(c, x)
+            self._parallel_two_norm_layers(c, x, x0)
         elif self.wiring == "streams":
             return self._logits(self._stream_layers(c, x, want_rows))
         for L in self.layers if self.wiring == "parallel" else ():
@@ -1208,35 +1353,41 @@ class HybridDecoder:
                                             _cabi.stream()), "pa_logit_softcap")
         return logits
 
-    def _parallel_two_norm_layers(self, c, x):
-        """x += mixer(N(x; w1)) + ff(N(x; w2)): both sublayers read the same x through norms that differ only in their
-        gains.  pa_residual_add_norm2 adds a layer's outputs to the float residual and leaves BOTH operands of the next
-        layer (one mean square) in the activation type."""
+    def _parallel_two_norm_layers(self, c, x, x0):
+        """x += mixer(N(x; w1)) + ff(N(x; w2)), over self.runs: both sublayers read the same x through norms that differ only
+        in their gains.  pa_residual_add_norm2_pass adds a layer's outputs to the float residual, then, in front of a looped
+        block's pass, x0 (the embedding output, not in the first pass) and the pass's step vector, and leaves BOTH operands of
+        the next layer (one mean square) in the activation type."""
         lib, R, W, s = self._lib, c.R, self.width, _cabi.stream()
 
-        def add_norm(add, nxt):
+        def add_norm(add, run):
             if add.get("shared") is not None:
                 raise ValueError("a shared expert is not served in the two-norm parallel wiring")
+            nxt, _mixer, t = run if run is not None else (None, None, None)
             h1 = c.empty(R, W) if nxt is not None else None
             h2 = c.empty(R, W) if nxt is not None and nxt.gain2 is not None else None
-            _chk(lib.pa_residual_add_norm2(x.data_ptr(), R, W, _cabi.ptr(add.get("y")), _cabi.ptr(add.get("dense")),
-                                           _cabi.ptr(add.get("routed")), _cabi.ptr(add.get("sel_w")),
-                                           _cabi.ptr(add.get("sel_id")), add.get("top", 0), add.get("experts", 0),
-                                           _cabi.ptr(add.get("ident")), self.eps,
-                                           _cabi.ptr(nxt.gain1) if nxt is not None else None, _cabi.ptr(h1),
-                                           _cabi.ptr(nxt.gain2) if h2 is not None else None, _cabi.ptr(h2), c.elem, s),
-                 "pa_residual_add_norm2")
+            if not add and nxt is None:
+                return None, None
+            _chk(lib.pa_residual_add_norm2_pass(
+                x.data_ptr(), R, W, _cabi.ptr(add.get("y")), _cabi.ptr(add.get("dense")), _cabi.ptr(add.get("routed")),
+                _cabi.ptr(add.get("sel_w")), _cabi.ptr(add.get("sel_id")), add.get("top", 0), add.get("experts", 0),
+                _cabi.ptr(add.get("ident")), _cabi.ptr(x0) if t else None,
+                _cabi.ptr(self.loop_step[t]) if t is not None else None, self.eps,
+                _cabi.ptr(nxt.gain1) if nxt is not None else None, _cabi.ptr(h1),
+                _cabi.ptr(nxt.gain2) if h2 is not None else None, _cabi.ptr(h2), c.elem, s), "pa_residual_add_norm2_pass")
             return h1, h2
 
-        layers = self.layers
-        h1, h2 = add_norm({}, layers[0]) if layers else (None, None)
-        for i, L in enumerate(layers):
-            add = dict(y=L.mixer.forward(c, h1))
+        runs = self.runs
+        h1, h2 = add_norm({}, runs[0]) if runs else (None, None)
+        for i, (L, mixer, _t) in enumerate(runs):
+            add = dict(y=mixer.forward(c, h1))
             if L.ff is not None:
                 add.update(L.ff.forward(c, h2))
-            h1, h2 = add_norm(add, layers[i + 1] if i + 1 < len(layers) else None)
-            if self.layer_hook is not None:
+            if self.layer_hook is not None:     # the residual as this layer leaves it, before what a pass starts with
+                add_norm(add, None)
+                add = {}
                 self.layer_hook(x)
+            h1, h2 = add_norm(add, runs[i + 1] if i + 1 < len(runs) else None)
 
     def _post_norm_layers(self, c, x):
         """x += N(mixer(x)), then x += N(ff(x)): the sublayers read the residual itself (rounded to the activation type

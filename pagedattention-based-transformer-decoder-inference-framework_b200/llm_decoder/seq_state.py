@@ -3,6 +3,8 @@
   * a STATE SLOT: one row in every per-layer float state tensor (the previous token's normalised row for token
     shift, a recurrent layer's hidden state, ...).  Slots come from a free list and are zeroed when handed out, so a
     new sequence starts from the all-zero state whatever the slot held before;
+  * its LAST TOKEN, for models whose embedding reads pairs of tokens (track_tokens): kept on the host, where the tokens
+    of a step arrive, and brought along as one more number per row;
   * its tiles in the paged K/V pools of the attention layers (one KVTileCache per layer, table row = slot), registered
     as its tokens arrive and released when it ends.
 
@@ -16,17 +18,19 @@ from .kv_tile_cache import KVTileCache
 
 
 class RaggedBatch:
-    """Device-side description of one step's rows (see csrc/seq_ops.cu): per row (slot, position, previous row or -1),
-    per portion (first row, length, slot).  Built by SequenceStateCache.make_batch."""
+    """Device-side description of one step's rows (see csrc/seq_ops.cu): per row (slot, position, previous row or -1,
+    and, where the model asks for it, the previous token or -1), per portion (first row, length, slot).  Built by SequenceStateCache.make_batch."""
 
-    def __init__(self, ids, row_slot, row_pos, row_prev, seq_start, seq_len, seq_slot, portions, device):
+    def __init__(self, ids, row_slot, row_pos, row_prev, seq_start, seq_len, seq_slot, portions, device, prev_ids=None):
         i32 = dict(dtype=torch.int32)
-        host = torch.from_numpy(np.stack([np.asarray(a, dtype=np.int32) for a in (ids, row_slot, row_pos, row_prev)]))
+        per_row = (ids, row_slot, row_pos, row_prev) + ((prev_ids,) if prev_ids is not None else ())
+        host = torch.from_numpy(np.stack([np.asarray(a, dtype=np.int32) for a in per_row]))
         self.rows = len(ids)
         self.num_seqs = len(seq_start)
         self.portions = portions                      # host list of (first row, length, slot, first position)
         dev_rows = _to_device(host, device)
         self.ids, self.row_slot, self.row_pos, self.row_prev = dev_rows[0], dev_rows[1], dev_rows[2], dev_rows[3]
+        self.prev_ids = dev_rows[4] if prev_ids is not None else None
         seqs = torch.tensor([seq_start, seq_len, seq_slot], **i32)
         dev_seqs = _to_device(seqs, device)
         self.seq_start, self.seq_len, self.seq_slot = dev_seqs[0], dev_seqs[1], dev_seqs[2]
@@ -76,6 +80,16 @@ class RaggedBatch:
             self._cache[key] = (t, len(items), b[0], b[1])
         return self._cache[key]
 
+    def portion_items(self, chunk):
+        """Every portion cut into runs of at most `chunk` consecutive tokens: ([n, 6] int32 device tensor of (first row,
+        tokens, slot, offset within the portion, the portion's length, first position), n)."""
+        key = ("pi", chunk)
+        if key not in self._cache:
+            items = [(r0 + o, min(chunk, n - o), slot, o, n, p0 + o) for r0, n, slot, p0 in self.portions for o in range(0, n, chunk)]
+            t = torch.tensor(items, dtype=torch.int32).reshape(-1, 6)
+            self._cache[key] = (_to_device(t, self.device), len(items))
+        return self._cache[key]
+
     def scan_chunks(self, chunk):
         """Chunk lists of the chunked recurrent scan: (chunk_start, chunk_len, seq_chunk0, seq_nchunks) device int32
         tensors and the chunk count."""
@@ -106,6 +120,8 @@ class SequenceStateCache:
         self._states = []           # float [max_seqs, width] tensors
         self._kv = []               # KVTileCache per attention layer
         self._len = {}              # slot -> tokens held
+        self.track_tokens = False   # batches carry the previous token of every row
+        self._last = {}             # slot -> last token (track_tokens)
 
     # ---- set-up (by the model, once) --------------------------------------------------------------------------------
     def add_state(self, width):
@@ -165,13 +181,14 @@ class SequenceStateCache:
         for kvc in self._kv:
             kvc.release_beam(slot)
         del self._len[slot]
+        self._last.pop(slot, None)
         self._free_slots.append(slot)
 
     # ---- batch description ------------------------------------------------------------------------------------------
     def make_batch(self, entries):
         """entries: [(slot, token ids)] in batch order, each slot at most once.  Extends every slot by its tokens and
         returns the RaggedBatch."""
-        ids, row_slot, row_pos, row_prev = [], [], [], []          # one int32 array per portion
+        ids, row_slot, row_pos, row_prev, prev_ids = [], [], [], [], []        # one int32 array (or list) per portion
         seq_start, seq_len, seq_slot, portions = [], [], [], []
         seen = set()
         r0 = 0
@@ -199,10 +216,15 @@ class SequenceStateCache:
                 prev = np.arange(r0 - 1, r0 + n - 1, dtype=np.int32)
                 prev[0] = -1
                 row_prev.append(prev)
+            if self.track_tokens:
+                before = self._last.get(slot, -1)
+                prev_ids.append([before] + ids[-1][:-1] if n < 16 else np.concatenate([[before], ids[-1][:-1]]).astype(np.int32))
+                self._last[slot] = int(ids[-1][-1])
             r0 += n
         def flat(pieces):
             if all(isinstance(a, list) for a in pieces):
                 return [v for a in pieces for v in a]
             return np.concatenate([np.asarray(a, dtype=np.int32) for a in pieces])
         ids, row_slot, row_pos, row_prev = flat(ids), flat(row_slot), flat(row_pos), flat(row_prev)
-        return RaggedBatch(ids, row_slot, row_pos, row_prev, seq_start, seq_len, seq_slot, portions, self.device)
+        return RaggedBatch(ids, row_slot, row_pos, row_prev, seq_start, seq_len, seq_slot, portions, self.device,
+                           flat(prev_ids) if self.track_tokens else None)
