@@ -33,6 +33,9 @@ extra  = the other BASELINE.json configurations under the same clock (benchmarks
          with convolved projections / sinks / a kept prefix / turned values, PolyNorm, identity experts) next to `Dubarax`.
 --namudra: likewise (benchmarks/namudra.py): the stack serving the `Namudra` design (residual streams, windowed sigmoid
          attention whose values are its keys, latent attention, rotated retention) next to `Dubarax` and `Domilix`.
+--tiradra: likewise (benchmarks/tiradra.py): the stack serving the `Tiradra` design (token-pair embedding, attention on
+         convolved / turned / normed projections, latent attention with sinks and an element gate) next to `Gunulorn` and
+         `Domilix`.
 N > 1: one process per GPU (torchrun), rows sharded across ranks, no data-path collective in the headline
          step; c5_splitkv is the mode with an exchange.
 """
@@ -88,6 +91,11 @@ def parse():
                          "the Namudra design at realistic layer sizes next to the Dubarax and Domilix designs at equal size, "
                          "and its kernels next to the like kernels of those designs against their rooflines "
                          "(benchmarks/namudra.py); one JSON line")
+    ap.add_argument("--tiradra", action="store_true",
+                    help="instead of the headline workload: prefill / decode throughput of the config-driven stack serving "
+                         "the Tiradra design at realistic layer sizes next to the Gunulorn and Domilix designs at equal size, "
+                         "and its kernels next to the like kernels of those designs against their rooflines "
+                         "(benchmarks/tiradra.py); one JSON line")
     ap.add_argument("--latent", action="store_true",
                     help="instead of the headline workload: prefill / decode throughput of the config-driven stack serving "
                          "the Domilix design (latent attention) at realistic layer sizes next to the Megusun design at "
@@ -481,6 +489,10 @@ def main():
     if args.namudra:
         from benchmarks import namudra
         print(json.dumps({"bench": "namudra", **namudra.run()}, default=float))
+        return
+    if args.tiradra:
+        from benchmarks import tiradra
+        print(json.dumps({"bench": "tiradra", **tiradra.run()}, default=float))
         return
     if args.latent:
         from benchmarks import latent
