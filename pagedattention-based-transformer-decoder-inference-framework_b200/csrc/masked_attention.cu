@@ -169,6 +169,7 @@ struct ConvAppendParams {
     const int32_t* items;       // [n][6]: first row, tokens, slot, offset within the portion, portion's length, first position
     int num_items;
     int pairs;                  // every pair of columns starts on a boundary of two elements
+    int words;                  // 4 or 8: heads are whole words of that many columns, everything aligned: the vector form
 };
 constexpr int kCaMaxTaps = 8;
 
@@ -334,6 +335,210 @@ __global__ void __launch_bounds__(256) conv_rope_norm_append_kernel(const ConvAp
     }
 }
 
+// The same for heads of at most 256 whose rows are whole words of EPL columns: a unit is LANES lanes with EPL neighbouring
+// columns each (the pairs of a rotation lie within a lane), 32 / LANES units per warp.  The raw rows of the next kAhead tokens
+// and the rotation of the next one are on their way while the current one is computed; the page of a row is looked up when a
+// new page begins.  The window is a ring of TAPS rows: the loop is unrolled over kAhead tokens (a multiple of TAPS), so
+// every place in it is fixed at compile time.
+constexpr int kCaThreads = 128;
+
+template <typename T, int EPL> struct CaWord { uint32_t w[EPL * sizeof(T) / 4]; };
+template <typename T, int EPL>
+__device__ __forceinline__ CaWord<T, EPL> ca_word_load(const T* __restrict__ p) {
+    CaWord<T, EPL> r;
+    if constexpr (EPL * sizeof(T) == 8) {
+        const uint2 v = *reinterpret_cast<const uint2*>(p);
+        r.w[0] = v.x; r.w[1] = v.y;
+    } else {
+#pragma unroll
+        for (int i = 0; i < (int)(EPL * sizeof(T) / 16); ++i) {
+            const uint4 v = reinterpret_cast<const uint4*>(p)[i];
+            r.w[4 * i] = v.x; r.w[4 * i + 1] = v.y; r.w[4 * i + 2] = v.z; r.w[4 * i + 3] = v.w;
+        }
+    }
+    return r;
+}
+template <typename T, int EPL>
+__device__ __forceinline__ void ca_word_unpack(const CaWord<T, EPL>& r, float (&f)[EPL]) {
+    if constexpr (sizeof(T) == 2) {
+#pragma unroll
+        for (int i = 0; i < EPL / 2; ++i) {
+            f[2 * i] = __uint_as_float(r.w[i] << 16);
+            f[2 * i + 1] = __uint_as_float(r.w[i] & 0xffff0000u);
+        }
+    } else {
+#pragma unroll
+        for (int i = 0; i < EPL; ++i) f[i] = __uint_as_float(r.w[i]);
+    }
+}
+template <typename T, int EPL>
+__device__ __forceinline__ void ca_word_store(T* __restrict__ p, const float (&f)[EPL]) {
+    if constexpr (sizeof(T) == 2 && EPL == 4) {
+        *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(f[0], f[1]), pack_bf16x2(f[2], f[3]));
+    } else if constexpr (sizeof(T) == 2) {
+        *reinterpret_cast<uint4*>(p) = bf16x8_pack(f);
+    } else {
+#pragma unroll
+        for (int i = 0; i < EPL / 4; ++i) reinterpret_cast<float4*>(p)[i] = make_float4(f[4 * i], f[4 * i + 1], f[4 * i + 2], f[4 * i + 3]);
+    }
+}
+template <int EPL>
+__device__ __forceinline__ void ca_load_floats(const float* __restrict__ p, float (&f)[EPL]) {
+#pragma unroll
+    for (int i = 0; i < EPL / 4; ++i) {
+        const float4 a = reinterpret_cast<const float4*>(p)[i];
+        f[4 * i] = a.x; f[4 * i + 1] = a.y; f[4 * i + 2] = a.z; f[4 * i + 3] = a.w;
+    }
+}
+
+template <typename T, int EPL, int LANES, int TAPS>
+__global__ void __launch_bounds__(kCaThreads, EPL == 4 && TAPS <= 4 ? 5 : 1) conv_rope_norm_append_vec_kernel(const ConvAppendParams p) {
+    constexpr int kAhead = TAPS < 4 ? 4 : TAPS;
+    const int lane = threadIdx.x & (LANES - 1);
+    const int units = p.heads + (p.k_pool ? 2 * p.kv_heads : 0);
+    const uint32_t uid = (blockIdx.x * (uint32_t)blockDim.x + threadIdx.x) / LANES;
+    // every lane of a warp stays to the end (the sums over a unit's lanes are warp shuffles); lanes past the last unit or past
+    // a head's size read its first columns and write nothing
+    const bool unit_ok = uid < (uint32_t)p.num_items * (uint32_t)units;
+    const int item = unit_ok ? (int)(uid / units) : 0, unit = unit_ok ? (int)(uid % units) : 0;
+    const int* it = p.items + 6 * item;
+    const int row0 = it[0], n = it[1], off = it[3], plen = it[4], pos0 = it[5];
+    const int kind = unit < p.heads ? 0 : unit < p.heads + p.kv_heads ? 1 : 2;       // query, key, value
+    const int g = kind == 0 ? 0 : unit - p.heads - (kind - 1) * p.kv_heads;
+    const int size = kind == 2 ? p.vdim : p.dim;
+    const bool slot_ok = (unsigned)it[2] < (unsigned)p.num_slots;
+    const bool live = unit_ok && lane * EPL < size && slot_ok;
+    const int slot = slot_ok ? it[2] : 0;
+    const int d = lane * EPL < size ? lane * EPL : 0;
+    const int ch0 = (kind == 0 ? unit * p.dim : p.heads * p.dim + (kind == 1 ? g * p.dim : p.kv_heads * p.dim + g * p.vdim)) + d;
+    const int stride = (int)p.in_stride;
+    const T* in = static_cast<const T*>(p.in) + p.in_off + ch0 + (int64_t)row0 * stride;
+    const int taps = p.w ? p.taps : 1;
+    float* st = taps > 1 ? p.state + (int64_t)slot * (taps - 1) * p.channels + ch0 : nullptr;
+    const int turned = kind < 2 ? min(EPL, max(0, p.rot_dims - d)) : 0;      // columns of this lane that are rotated
+    const float* rp = p.rope + (int64_t)row0 * p.rot_dims + d;
+    const bool norm = kind < 2 && p.norm;
+    const float inv_size = 1.0f / (float)size;
+
+    CaWord<T, EPL> nxt[kAhead];
+#pragma unroll
+    for (int i = 0; i < kAhead; ++i) nxt[i] = ca_word_load<T, EPL>(in + (int64_t)min(i, n - 1) * stride);
+    float cs[EPL];                                     // cos, sin of this lane's pairs at the current token
+#pragma unroll
+    for (int c = 0; c < EPL; ++c) cs[c] = 0.f;
+    auto load_turn = [&]() {
+#pragma unroll
+        for (int c = 0; c < EPL; c += 4)
+            if (c < turned) {
+                const float4 v = *reinterpret_cast<const float4*>(rp + c);
+                cs[c] = v.x; cs[c + 1] = v.y; cs[c + 2] = v.z; cs[c + 3] = v.w;
+            }
+        rp += p.rot_dims;
+    };
+    load_turn();
+    float wt[TAPS][EPL], win[TAPS][EPL];               // win: ring, token t in place t % TAPS
+#pragma unroll
+    for (int b = 0; b < TAPS; ++b)
+#pragma unroll
+        for (int c = 0; c < EPL; ++c) {
+            wt[b][c] = p.w ? 0.f : b == 0 ? 1.f : 0.f;
+            win[b][c] = 0.f;
+        }
+    if (p.w) {
+#pragma unroll
+        for (int b = 0; b < TAPS; ++b)
+            if (b < taps) ca_load_floats<EPL>(p.w + (int64_t)b * p.channels + ch0, wt[b]);
+    }
+#pragma unroll
+    for (int b = 1; b < TAPS; ++b)
+        if (b < taps) {
+            const int t = off - b;                     // offset within the portion
+            if (t >= 0) ca_word_unpack<T, EPL>(ca_word_load<T, EPL>(in - (int64_t)b * stride), win[TAPS - b]);
+            else ca_load_floats<EPL>(st + (int64_t)(taps - 1 + t) * p.channels, win[TAPS - b]);
+        }
+    // destination of the current token's row (null: not stored), and its place in its page
+    T* dst = kind == 0 ? static_cast<T*>(p.q_out) + (int64_t)row0 * p.q_out_stride + ch0 : nullptr;
+    const int64_t dstep = kind == 0 ? p.q_out_stride : size;
+    int tile = 0, at = 0;
+    auto look_up = [&]() {
+        const int page = tile < p.num_tiles ? p.table[((int64_t)slot * p.kv_heads + g) * p.num_tiles + tile] : -1;
+        dst = page >= 0 && page < p.total_pages
+                  ? static_cast<T*>(kind == 1 ? p.k_pool : p.v_pool) + ((int64_t)page * p.tile_size + at) * size + d : nullptr;
+    };
+    if (kind && pos0 >= 0) {
+        tile = pos0 / p.tile_size;
+        at = pos0 - tile * p.tile_size;
+        look_up();
+    }
+
+    for (int t0 = 0; t0 < n; t0 += kAhead) {         // units of a warp with fewer tokens leave the loop as a whole
+#pragma unroll
+        for (int i = 0; i < kAhead; ++i) {
+            const int t = t0 + i;
+            if (t >= n) break;
+            float y[EPL];
+            float (&now)[EPL] = win[i % TAPS];
+            ca_word_unpack<T, EPL>(nxt[i], now);
+            if (t + kAhead < n) nxt[i] = ca_word_load<T, EPL>(in + (int64_t)(t + kAhead) * stride);
+#pragma unroll
+            for (int c = 0; c < EPL; ++c) {
+                y[c] = wt[0][c] * now[c];
+#pragma unroll
+                for (int b = 1; b < TAPS; ++b) y[c] = fmaf(wt[b][c], win[(i + TAPS - b) % TAPS][c], y[c]);
+            }
+#pragma unroll
+            for (int c = 0; c < EPL; c += 4)
+                if (c < turned) {
+                    const float u0 = y[c], v0 = y[c + 1], u1 = y[c + 2], v1 = y[c + 3];
+                    y[c] = u0 * cs[c] - v0 * cs[c + 1];
+                    y[c + 1] = v0 * cs[c] + u0 * cs[c + 1];
+                    y[c + 2] = u1 * cs[c + 2] - v1 * cs[c + 3];
+                    y[c + 3] = v1 * cs[c + 2] + u1 * cs[c + 3];
+                }
+            if (t + 1 < n) load_turn();
+            if (norm) {
+                float ss = 0.f;
+#pragma unroll
+                for (int c = 0; c < EPL; ++c) ss = fmaf(y[c], y[c], ss);
+                if (lane * EPL >= size) ss = 0.f;
+                const unsigned mask = LANES == 32 ? 0xffffffffu : ((1u << LANES) - 1u) << (threadIdx.x & 31 & ~(LANES - 1));
+#pragma unroll
+                for (int o = LANES / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(mask, ss, o);
+                const float rn = rsqrtf(fmaf(ss, inv_size, p.eps));
+#pragma unroll
+                for (int c = 0; c < EPL; ++c) y[c] *= rn;
+            }
+            if (live && dst) ca_word_store<T, EPL>(dst, y);
+            if (dst) dst += dstep;
+            if (kind && ++at == p.tile_size) {
+                at = 0;
+                ++tile;
+                if (t + 1 < n) look_up();
+            }
+        }
+    }
+
+    if (!live || off != 0 || taps <= 1) return;
+    for (int j = 0; j < taps - 1; ++j) {               // rows older than the portion move up within the slot
+        const int t = plen - (taps - 1) + j;
+        float f[EPL];
+        if (t >= 0) ca_word_unpack<T, EPL>(ca_word_load<T, EPL>(in + (int64_t)t * stride), f);
+        else ca_load_floats<EPL>(st + (int64_t)(taps - 1 + t) * p.channels, f);
+        ca_word_store<float, EPL>(st + (int64_t)j * p.channels, f);
+    }
+}
+
+template <typename T, int EPL, int LANES>
+static int ca_launch_vec(const ConvAppendParams& p, cudaStream_t st) {
+    const int units = p.heads + (p.k_pool ? 2 * p.kv_heads : 0);
+    const unsigned grid = (unsigned)(((int64_t)p.num_items * units * LANES + kCaThreads - 1) / kCaThreads);
+    const int taps = p.w ? p.taps : 1;
+    if (taps <= 1) conv_rope_norm_append_vec_kernel<T, EPL, LANES, 1><<<grid, kCaThreads, 0, st>>>(p);
+    else if (taps <= 4) conv_rope_norm_append_vec_kernel<T, EPL, LANES, 4><<<grid, kCaThreads, 0, st>>>(p);
+    else conv_rope_norm_append_vec_kernel<T, EPL, LANES, kCaMaxTaps><<<grid, kCaThreads, 0, st>>>(p);
+    PA_RETURN_LAUNCH_STATUS();
+}
+
 template <typename T, int NP>
 static int ca_launch(const ConvAppendParams& p, cudaStream_t st) {
     const int units = p.heads + (p.k_pool ? 2 * p.kv_heads : 0);
@@ -348,6 +553,12 @@ static int ca_launch(const ConvAppendParams& p, cudaStream_t st) {
 template <typename T>
 static int ca_dispatch(const ConvAppendParams& p, cudaStream_t st) {
     const int n = p.k_pool && p.vdim > p.dim ? p.vdim : p.dim;
+    if (p.words >= 4 && n <= 128) {
+        if (n <= 32) return ca_launch_vec<T, 4, 8>(p, st);
+        if (n <= 64) return ca_launch_vec<T, 4, 16>(p, st);
+        return ca_launch_vec<T, 4, 32>(p, st);
+    }
+    if (p.words == 8 && n <= 256) return ca_launch_vec<T, 8, 32>(p, st);
     if (n <= 64) return ca_launch<T, 1>(p, st);
     if (n <= 128) return ca_launch<T, 2>(p, st);
     if (n <= 256) return ca_launch<T, 4>(p, st);
@@ -1552,6 +1763,15 @@ PA_API int pa_conv_rope_norm_append(const void* d_in, int64_t in_stride, int in_
     const uintptr_t two = 2 * (uintptr_t)(elem == 2 ? 2 : 4);
     p.pairs = dim % 2 == 0 && vdim % 2 == 0 && in_stride % 2 == 0 && in_off % 2 == 0 && q_out_stride % 2 == 0 &&
               ((uintptr_t)d_in | (uintptr_t)d_q_out | (uintptr_t)d_k_pool | (uintptr_t)d_v_pool) % two == 0;
+    // the vector form: columns in words of four or eight, 32-bit unit numbers
+    auto words = [&](int k) {
+        const uintptr_t bytes = (uintptr_t)(k * (elem == 2 ? 2 : 4) < 16 ? k * 2 : 16);
+        return dim % k == 0 && vdim % k == 0 && in_stride % k == 0 && in_off % k == 0 && q_out_stride % k == 0 &&
+               ((uintptr_t)d_in | (uintptr_t)d_q_out | (uintptr_t)d_k_pool | (uintptr_t)d_v_pool) % bytes == 0;
+    };
+    const bool floats = ((uintptr_t)d_weight | (uintptr_t)d_state | (uintptr_t)d_rope) % 16 == 0 && rot_dims % 4 == 0;
+    const bool small = (int64_t)num_items * (heads + 2 * kv_heads) < (1 << 26) && in_stride < (1 << 30);
+    p.words = !floats || !small ? 0 : words(8) ? 8 : words(4) ? 4 : 0;
     if (elem == 4) return ca_dispatch<float>(p, as_stream(stream));
     if (elem == 2) return ca_dispatch<bf16_t>(p, as_stream(stream));
     return PA_ERR_UNSUPPORTED;

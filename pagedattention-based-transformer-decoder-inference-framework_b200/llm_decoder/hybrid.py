@@ -587,6 +587,8 @@ class MaskedAttention:
                 raise ValueError(f"{prefix}: rot.dims must be even and at most dim")
         if self.rot_values and self.vdim % 2:
             raise ValueError(f"{prefix}: turned values need an even vdim")
+        # everything between the input product and the attention in one launch, where the layer has nothing that launch lacks
+        self.fused_append = self.turned_norm or (self.taps > 0 and not self.rot_values and not self.qk_norm and self.dim <= 512 and self.vdim <= 512)
         self.head_scale = None
         if head_temp:
             if tuple(W[prefix + "temp"].shape) != (H,):
@@ -647,15 +649,16 @@ class MaskedAttention:
         """Convolution and rotation of this step's q | k | v rows, then the new keys and values go to the pool.  Returns
         the buffer and column offset the attention kernels read the queries from."""
         b, lib, s, R = c.batch, c.lib, _cabi.stream(), c.R
-        if self.turned_norm:        # convolution, rotation, norm and append: one launch
-            kv, pt = self.kv, self.kv.page_table_
+        if self.fused_append:       # convolution, rotation, norm and append: one launch
+            kv, pt, own = self.kv, self.kv.page_table_, self.own_kv
             items, n = b.portion_items(APPEND_CHUNK)
             q = c.empty(R, self.q_cols)
             _chk(lib.pa_conv_rope_norm_append(
                 proj.data_ptr(), proj.stride(0), off, self.heads, self.kv_heads, self.dim, self.vdim, self.taps,
                 _cabi.ptr(self.conv_wt) if self.taps else None, _cabi.ptr(self.conv_state), self.rot_dims,
-                _cabi.ptr(c.rope_table(self.rot_dims, self.rot_base, self.rot_scaling)), 1, c.model.eps, q.data_ptr(), self.q_cols,
-                kv.key_buffer_.data_ptr(), kv.value_buffer_.data_ptr(), pt.device_data().data_ptr(), pt.num_beams_,
+                _cabi.ptr(c.rope_table(self.rot_dims, self.rot_base, self.rot_scaling)),
+                1 if self.turned_norm else 0, c.model.eps, q.data_ptr(), self.q_cols, kv.key_buffer_.data_ptr() if own else None,
+                kv.value_buffer_.data_ptr() if own else None, pt.device_data().data_ptr(), pt.num_beams_,
                 pt.num_tiles_, kv.total_pages_, kv.tile_size_, items.data_ptr(), n, APPEND_CHUNK, c.elem, s),
                 "pa_conv_rope_norm_append")
             return q, 0

@@ -71,6 +71,14 @@ class KVTileCache:
     def configure_table(self, num_beams, num_heads, num_tiles):
         self.page_table_.init(num_beams, num_heads, num_tiles)
 
+    def share_pages(self, owner):
+        """Pages of this pool are those of `owner` (a pool of as many pages and tokens per page): one page table, one free list,
+        one registration per tile serve both, each with rows of its own."""
+        if (self.total_pages_, self.tile_size_) != (owner.total_pages_, owner.tile_size_):
+            raise ValueError("KVTileCache.share_pages: the pools differ in pages or tile size")
+        self.page_table_, self.tile_to_page_map_, self._free = owner.page_table_, owner.tile_to_page_map_, owner._free
+        self._page_refs, self.mutex_ = owner._page_refs, owner.mutex_
+
     def _dev(self):
         return self._device or torch.device("cuda", torch.cuda.current_device())
 

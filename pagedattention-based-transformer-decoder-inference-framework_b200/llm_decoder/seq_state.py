@@ -6,7 +6,8 @@
   * its LAST TOKEN, for models whose embedding reads pairs of tokens (track_tokens): kept on the host, where the tokens
     of a step arrive, and brought along as one more number per row;
   * its tiles in the paged K/V pools of the attention layers (one KVTileCache per layer, table row = slot), registered
-    as its tokens arrive and released when it ends.
+    as its tokens arrive and released when it ends.  Layers with equally many key/value heads hold a request's tiles in the
+    same pages of their pools, so they share ONE page table and one registration per tile.
 
 The pools are sized for `max_tokens` live tokens (each request rounded up to whole tiles), not for the sum of all
 requests: pages and slots are used again, and running out is an error, never an eviction of a live request."""
@@ -15,6 +16,29 @@ import torch
 
 from .host_stage import to_device as _to_device
 from .kv_tile_cache import KVTileCache
+
+
+def _runs(portions, step):
+    """Every portion (first row, length, slot, first position) cut into runs of at most `step` consecutive tokens (0: whole
+    portions), in portion order: an int32 array [n, 6] of (first row, tokens, slot, offset within the portion, the portion's
+    length, first position)."""
+    pieces, short = [], []
+    for r0, n, slot, p0 in portions:
+        if step <= 0 or n <= step:
+            short.append((r0, n, slot, 0, n, p0))
+        elif n <= 4 * step:         # a few runs: plain tuples cost less than an array
+            short.extend((r0 + o, min(step, n - o), slot, o, n, p0 + o) for o in range(0, n, step))
+        else:
+            if short:
+                pieces.append(np.array(short, dtype=np.int32))
+                short = []
+            o = np.arange(0, n, step, dtype=np.int32)
+            a = np.empty((len(o), 6), dtype=np.int32)
+            a[:, 0], a[:, 1], a[:, 2], a[:, 3], a[:, 4], a[:, 5] = r0 + o, np.minimum(step, n - o), slot, o, n, p0 + o
+            pieces.append(a)
+    if short:
+        pieces.append(np.array(short, dtype=np.int32))
+    return pieces[0] if len(pieces) == 1 else np.concatenate(pieces)
 
 
 class RaggedBatch:
@@ -46,20 +70,20 @@ class RaggedBatch:
         key = ("qt", tile_tokens, big_tokens, big_from)
         if key not in self._cache:
             groups = {0: [], 1: [], 2: []}
-            for r0, n, slot, p0 in self.portions:
-                kind = 1 if n == 1 else 2 if big_tokens and n >= big_from else 0
-                step = big_tokens if kind == 2 else tile_tokens
-                for o in range(0, n, step):
-                    groups[kind].append((r0 + o, min(step, n - o), slot, p0 + o))
+            for p in self.portions:
+                groups[1 if p[1] == 1 else 2 if big_tokens and p[1] >= big_from else 0].append(p)
             out = {}
-            for kind, tiles in groups.items():
-                if not tiles:
+            for kind, portions in groups.items():
+                if not portions:
                     out[kind] = None
                     continue
-                t = torch.tensor(tiles, dtype=torch.int32).reshape(-1, 4)
-                out[kind] = (_to_device(t, self.device), len(tiles), max(p + m for _r, m, _s, p in tiles))
+                runs = _runs(portions, big_tokens if kind == 2 else tile_tokens)
+                out[kind] = (self._upload(runs[:, [0, 1, 2, 5]]), len(runs), int((runs[:, 5] + runs[:, 1]).max()))
             self._cache[key] = out
         return self._cache[key]
+
+    def _upload(self, array):
+        return _to_device(torch.from_numpy(np.ascontiguousarray(array)), self.device)
 
     def chunk_items(self, chunk):
         """Every portion cut into runs of at most `chunk` consecutive tokens (0: whole portions), in portion order, as work
@@ -67,17 +91,11 @@ class RaggedBatch:
         offset of the first token within its portion), n, first item per portion, items per portion)."""
         key = ("ci", chunk)
         if key not in self._cache:
-            items, s0, sn = [], [], []
-            for r0, n, slot, _p0 in self.portions:
-                s0.append(len(items))
-                step = chunk if chunk > 0 else n
-                for o in range(0, n, step):
-                    items.append((r0 + o, min(step, n - o), slot, o))
-                sn.append(len(items) - s0[-1])
-            t = torch.tensor(items, dtype=torch.int32).reshape(-1, 4)
-            b = torch.tensor([s0, sn], dtype=torch.int32)
-            t, b = _to_device(t, self.device), _to_device(b, self.device)
-            self._cache[key] = (t, len(items), b[0], b[1])
+            runs = _runs(self.portions, chunk)
+            starts = np.flatnonzero(runs[:, 3] == 0).astype(np.int32)
+            counts = np.diff(starts, append=np.int32(len(runs)))
+            b = self._upload(np.stack([starts, counts]))
+            self._cache[key] = (self._upload(runs[:, :4]), len(runs), b[0], b[1])
         return self._cache[key]
 
     def portion_items(self, chunk):
@@ -85,9 +103,8 @@ class RaggedBatch:
         tokens, slot, offset within the portion, the portion's length, first position), n)."""
         key = ("pi", chunk)
         if key not in self._cache:
-            items = [(r0 + o, min(chunk, n - o), slot, o, n, p0 + o) for r0, n, slot, p0 in self.portions for o in range(0, n, chunk)]
-            t = torch.tensor(items, dtype=torch.int32).reshape(-1, 6)
-            self._cache[key] = (_to_device(t, self.device), len(items))
+            runs = _runs(self.portions, chunk)
+            self._cache[key] = (self._upload(runs), len(runs))
         return self._cache[key]
 
     def scan_chunks(self, chunk):
@@ -119,6 +136,7 @@ class SequenceStateCache:
         self._free_slots = list(range(self.max_seqs - 1, -1, -1))
         self._states = []           # float [max_seqs, width] tensors
         self._kv = []               # KVTileCache per attention layer
+        self._tables = []           # the ones among them that hand out pages: one per count of key/value heads
         self._len = {}              # slot -> tokens held
         self.track_tokens = False   # batches carry the previous token of every row
         self._last = {}             # slot -> last token (track_tokens)
@@ -130,12 +148,17 @@ class SequenceStateCache:
         return t
 
     def add_kv_layer(self, kv_heads, key_dim, value_dim, dtype, key_scale=False):
-        """A paged pool for one attention layer: max_tiles * kv_heads pages; the table has one row per slot and lets a
-        single request grow to the whole pool.  key_scale: a float per key beside the pool (key_scale_, by pool row)."""
+        """A paged pool for one attention layer: max_tiles * kv_heads pages; the table (shared by the layers with as many
+        heads) has one row per slot and lets a single request grow to the whole pool.  key_scale: a float per key beside the pool (key_scale_, by pool row)."""
         kvc = KVTileCache(dtype, device=self.device)
         kvc.init(self.max_tiles * int(kv_heads), self.tile_size, int(key_dim), int(value_dim))
-        kvc.configure_table(self.max_seqs, int(kv_heads), self.max_tiles)
         kvc.evict_on_exhaustion = False
+        owner = next((k for k in self._tables if k.page_table_.num_heads_ == int(kv_heads)), None)
+        if owner is None:
+            kvc.configure_table(self.max_seqs, int(kv_heads), self.max_tiles)
+            self._tables.append(kvc)
+        else:
+            kvc.share_pages(owner)
         kvc.key_scale_ = None
         if key_scale:
             kvc.key_scale_ = torch.zeros(kvc.total_pages_ * self.tile_size, dtype=torch.float32, device=self.device)
@@ -162,7 +185,7 @@ class SequenceStateCache:
         """Tokens that can still be taken (whole free tiles)."""
         if not self._kv:
             return 1 << 60
-        return min(k.free_pages() // k.page_table_.num_heads_ for k in self._kv) * self.tile_size
+        return min(k.free_pages() // k.page_table_.num_heads_ for k in self._tables) * self.tile_size
 
     def extend(self, slot, n_new):
         """Reserve room for the next n_new tokens of `slot`: registers the tiles they touch in every attention layer's
@@ -172,13 +195,13 @@ class SequenceStateCache:
         t1 = (pos0 + n_new + self.tile_size - 1) // self.tile_size
         if t1 > self.max_tiles:
             raise RuntimeError("SequenceStateCache: request exceeds the pool")
-        for kvc in self._kv:
+        for kvc in self._tables:
             kvc.register_range(slot, t0, t1)
         self._len[slot] = pos0 + n_new
         return pos0
 
     def free(self, slot):
-        for kvc in self._kv:
+        for kvc in self._tables:
             kvc.release_beam(slot)
         del self._len[slot]
         self._last.pop(slot, None)

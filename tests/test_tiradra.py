@@ -401,6 +401,7 @@ def test_slots_and_pages_are_used_again():
     config, W = _case("full")
     model = _model(config, W, max_tokens=160, max_seqs=2)
     assert len(model.states._kv) == 2 * 3 + 2               # the three looped layers have a pool per pass
+    assert len(model.states._tables) == 3                   # layers with one, two and three key/value heads share a page table each
     eng = ld.Engine(model)
     seqs = [_tokens(n, config["vocab"], 20 + i) for i, n in enumerate([90, 60, 33, 100, 17, 59])]
     out = eng.step([("r0", seqs[0][:50], list(range(50))), ("r1", seqs[1][:10], list(range(10)))])
